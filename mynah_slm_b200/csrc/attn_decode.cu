@@ -36,6 +36,9 @@ struct DecodeArgs {
     float softcap;       // 0: none; c: score <- c * tanh(score / c), after the scale
     int keep_first;      // with a window: keys at positions below it stay visible whatever their distance
     int vdiv;            // kv head g reads value head g / vdiv
+    int null_key;        // 1: the softmax has one more term, of score 0 and without a value
+    float out_scale;     // factor on the output rows
+    int vdo;             // columns of a head in the output rows (<= VD)
 };
 
 // The pages that the query of a sequence of `hi` positions can see: pages [pg0, pg1) of the window (or of everything),
@@ -213,7 +216,8 @@ attn_decode_split_kernel(const T* __restrict__ q, const T* __restrict__ k_cache,
 template <typename T>
 __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                            T* __restrict__ out, const int* __restrict__ kv_len, int window, int chunk,
-                                           int keep_first, int H, int HD, int S_max, int ldo) {
+                                           int keep_first, int H, int HD, int S_max, int ldo, int null_key, float out_scale,
+                                           int vdo) {
     const int h = blockIdx.x, b = blockIdx.y;
     const size_t row0 = ((size_t)b * H + h) * S_max;
     // only the pages the sequence can see have partial results
@@ -226,14 +230,15 @@ __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o, con
         const float m = part_ml[(row0 + s) * 2];
         ls += mn == -INFINITY ? 0.f : part_ml[(row0 + s) * 2 + 1] * expf(m - mn);
     }
-    const float inv = ls > 0.f ? 1.0f / ls : 0.f;
-    for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+    if (null_key && ls > 0.f) ls += expf(-mn);         // the term without a key; where it overflows the keys' share is zero
+    const float inv = ls > 0.f ? out_scale / ls : 0.f;
+    for (int d = threadIdx.x; d < vdo; d += blockDim.x) {
         float os = 0.f;
         for (int s = 0; s < S; s++) {
             const float m = part_ml[(row0 + s) * 2];
             if (m != -INFINITY) os += part_o[(row0 + s) * HD + d] * expf(m - mn);
         }
-        out[(size_t)b * ldo + (size_t)h * HD + d] = from_f32<T>(os * inv);
+        out[(size_t)b * ldo + (size_t)h * vdo + d] = from_f32<T>(os * inv);
     }
 }
 
@@ -256,7 +261,8 @@ int launch_decode(const void* q, void* out, int B, const DecodeArgs& a, const vo
         attn_decode_split_kernel<T, 4><<<grid, WARPS * 32, 0, stream>>>(qp, kp, vp, kv_len, pt, a, part_o, part_ml, status);
     if (mynah_check_launch("attn_decode_split")) return -1;
     const int threads = a.VD >= 128 ? 128 : (a.VD >= 64 ? 64 : 32);
-    attn_decode_combine_kernel<T><<<dim3(a.H, B), threads, 0, stream>>>(part_o, part_ml, (T*)out, kv_len, a.window, a.chunk, a.keep_first, a.H, a.VD, a.S, a.ldo);
+    attn_decode_combine_kernel<T><<<dim3(a.H, B), threads, 0, stream>>>(part_o, part_ml, (T*)out, kv_len, a.window, a.chunk, a.keep_first, a.H, a.VD, a.S, a.ldo,
+                                                                        a.null_key, a.out_scale, a.vdo);
     return mynah_check_launch("attn_decode_combine");
 }
 
@@ -289,13 +295,14 @@ MYNAH_API int mynah_attn_decode(
 }
 
 // The same with capped scores (softcap c > 0: score <- c tanh(score / c)), first tokens that a window keeps
-// (keep_first) and several key heads on one value head (the value cache has KV / vdiv heads).
+// (keep_first), several key heads on one value head (the value cache has KV / vdiv heads), one more softmax term of score
+// 0 that has no value (null_key), a factor on the output (out_scale) and output heads of `vdo` columns (0: VD).
 MYNAH_API int mynah_attn_decode_capped(
     const void* q, void* out, int dtype, int B, int H, int KV, int HD, int VD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int n_splits, float* scratch, int* status,
-    cudaStream_t stream);
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, float out_scale, int vdo,
+    int n_splits, float* scratch, int* status, cudaStream_t stream);
 
 MYNAH_API int mynah_attn_decode_ex(
     const void* q, void* out, int dtype, int B, int H, int KV, int HD, int VD, int ldq, int ldo,
@@ -303,21 +310,22 @@ MYNAH_API int mynah_attn_decode_ex(
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
     int window, int chunk, float scale, int n_splits, float* scratch, int* status, cudaStream_t stream) {
     return mynah_attn_decode_capped(q, out, dtype, B, H, KV, HD, VD, ldq, ldo, k_cache, v_cache, kv_len, page_indptr, page_ids,
-                                    page_base, n_pages, window, chunk, scale, 0.f, 0, 1, n_splits, scratch, status, stream);
+                                    page_base, n_pages, window, chunk, scale, 0.f, 0, 1, 0, 1.0f, VD, n_splits, scratch, status, stream);
 }
 
 MYNAH_API int mynah_attn_decode_capped(
     const void* q, void* out, int dtype, int B, int H, int KV, int HD, int VD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int n_splits, float* scratch, int* status,
-    cudaStream_t stream) {
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, float out_scale, int vdo,
+    int n_splits, float* scratch, int* status, cudaStream_t stream) {
     if (B == 0) return 0;
     MYNAH_REQUIRE(softcap >= 0.f && keep_first >= 0 && vdiv >= 1 && KV % vdiv == 0, "attn_decode: bad cap, kept tokens or value sharing");
     MYNAH_REQUIRE(keep_first == 0 || chunk == 0, "attn_decode: kept first tokens and a chunk mask do not go together");
     MYNAH_REQUIRE(B > 0 && H > 0 && KV > 0 && HD > 0 && H % KV == 0, "attn_decode: bad sizes B=%d H=%d KV=%d HD=%d", B, H, KV, HD);
     MYNAH_REQUIRE(HD % 8 == 0 && HD <= 256, "attn_decode: head_dim %d must be a multiple of 8 and at most 256", HD);
     MYNAH_REQUIRE(VD > 0 && VD % 8 == 0 && VD <= 256, "attn_decode: a value head of %d must be a multiple of 8 and at most 256", VD);
+    MYNAH_REQUIRE(vdo >= 0 && vdo <= VD, "attn_decode: %d output columns a head exceed the value head of %d", vdo, VD);
     MYNAH_REQUIRE(chunk >= 0, "attn_decode: negative chunk");
     MYNAH_REQUIRE(ldq % 8 == 0, "attn_decode: query row stride %d must be a multiple of 8", ldq);
     MYNAH_REQUIRE(n_splits >= 1 && n_splits <= 65535, "attn_decode: bad split count %d", n_splits);
@@ -325,7 +333,8 @@ MYNAH_API int mynah_attn_decode_capped(
     MYNAH_REQUIRE(scratch != nullptr, "attn_decode: no scratch memory given");
     int lpk = 1;
     while (lpk * 8 < HD || lpk * 8 < VD) lpk <<= 1;
-    const DecodeArgs a{H, KV, HD, ldq, ldo, window, n_splits, lpk, scale != 0.f ? scale : 1.0f / sqrtf((float)HD), VD, chunk, softcap, keep_first, vdiv};
+    const DecodeArgs a{H, KV, HD, ldq, ldo, window, n_splits, lpk, scale != 0.f ? scale : 1.0f / sqrtf((float)HD), VD, chunk, softcap, keep_first, vdiv,
+                       null_key, out_scale, vdo > 0 ? vdo : VD};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     float* part_o = scratch;
     float* part_ml = scratch + (size_t)B * H * n_splits * VD;

@@ -67,6 +67,9 @@ struct TcArgs {
                             // lists must then hold every page of a sequence
     int vdiv = 1;           // kv head g reads value head g / vdiv (the value cache has KV / vdiv heads)
     float softcap = 0.f;    // c > 0: score <- c tanh(score / c), after the scale
+    int null_key = 0;       // 1: the softmax has one more term, of score 0 and without a value (the merge adds it)
+    float out_scale = 1.f;  // factor on the output rows
+    int vdo = 0;            // columns of a head in the output rows; 0: the value head's width
 };
 
 // The pages that a sequence's newest position sees: pages [pg0, pg1) of its window (or of everything), and before them
@@ -174,20 +177,20 @@ __device__ __forceinline__ void write_empty_partial(const PageJob& j, const TcAr
 }
 
 // The page's K tile, then its V tile, each as its own copy group. Rows that are not visible are zero-filled.
-template <int HD>
+template <int HD, int VD = HD>
 __device__ __forceinline__ void issue_page_copies(const PageJob& j, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
                                                   const TcArgs& a, uint32_t k_base, uint32_t v_base) {
-    constexpr int CH = HD / 8;
+    constexpr int CH = HD / 8, VCH = VD / 8;
     const bf16* k_src = k_cache + ((size_t)j.page * a.KV + j.g) * PAGE_TOKENS * HD;
-    const bf16* v_src = v_cache + ((size_t)j.page * (a.KV / a.vdiv) + j.g / a.vdiv) * PAGE_TOKENS * HD;
+    const bf16* v_src = v_cache + ((size_t)j.page * (a.KV / a.vdiv) + j.g / a.vdiv) * PAGE_TOKENS * VD;
     for (int i = threadIdx.x; i < KEYS * CH; i += blockDim.x) {
         const int r = i / CH, c = i % CH;
         cp_async_16(k_base + swz<CH>(r, c), k_src + (size_t)r * HD + c * 8, j.sees(r));
     }
     cp_async_commit();
-    for (int i = threadIdx.x; i < KEYS * CH; i += blockDim.x) {
-        const int r = i / CH, c = i % CH;
-        cp_async_16(v_base + swz<CH>(r, c), v_src + (size_t)r * HD + c * 8, j.sees(r));
+    for (int i = threadIdx.x; i < KEYS * VCH; i += blockDim.x) {
+        const int r = i / VCH, c = i % VCH;
+        cp_async_16(v_base + swz<VCH>(r, c), v_src + (size_t)r * VD + c * 8, j.sees(r));
     }
     cp_async_commit();
 }
@@ -214,12 +217,12 @@ __device__ __forceinline__ void load_q_fragments(const PageJob& j, const bf16* _
 // [16 ks, 16 ks + 16) for this warp's n-tiles nt and nt + 1; before_k() and before_v() run before the first use of
 // each (waits and barriers, if the fragments still lie in shared memory). The arithmetic, and so every bit of the
 // result, is the same whoever provides them.
-template <int HD, class SYNC, class KFRAG, class VFRAG, class BEFORE_K, class BEFORE_V>
+template <int HD, int VD, class SYNC, class KFRAG, class VFRAG, class BEFORE_K, class BEFORE_V>
 __device__ __forceinline__ void compute_page_core(const PageJob& job, const uint32_t (&qa)[HD / 16][4], const TcArgs& a,
                                                   KFRAG k_frag, VFRAG v_frag, BEFORE_K before_k, BEFORE_V before_v,
                                                   bf16* p_s, float (*red_m)[MAX_G], float (*red_l)[MAX_G],
                                                   float* __restrict__ part_o, float* __restrict__ part_ml) {
-    constexpr int KSTEPS = HD / 16, NT = HD / 32;
+    constexpr int KSTEPS = HD / 16, NT = VD / 32;
     const int G = a.H / a.KV;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int k_first = job.k_first, k_last = job.k_last;
@@ -290,7 +293,7 @@ __device__ __forceinline__ void compute_page_core(const PageJob& job, const uint
     }
     before_v();                                       // (a barrier: the probabilities and the sums are in shared memory)
 
-    // ---- output: warp w takes dims [w*HD/4, (w+1)*HD/4): HD/32 n-tiles of 8, four k-steps of 16 keys
+    // ---- output: warp w takes dims [w*VD/4, (w+1)*VD/4): VD/32 n-tiles of 8, four k-steps of 16 keys
     float oc[NT][4] = {};
     {
         const uint32_t p_base = smem_u32(p_s);
@@ -315,10 +318,10 @@ __device__ __forceinline__ void compute_page_core(const PageJob& job, const uint
     for (int j = 0; j < 2; j++) {
         const int h = hrow + 8 * j;
         if (h < G) {
-            float* o = part_o + (row0 + (size_t)h * a.S) * HD;
+            float* o = part_o + (row0 + (size_t)h * a.S) * VD;
 #pragma unroll
             for (int nt = 0; nt < NT; nt++) {
-                const int d = warp * (HD / 4) + nt * 8 + (lane & 3) * 2;
+                const int d = warp * (VD / 4) + nt * 8 + (lane & 3) * 2;
                 *reinterpret_cast<float2*>(o + d) = make_float2(oc[nt][2 * j], oc[nt][2 * j + 1]);
             }
         }
@@ -350,14 +353,14 @@ __device__ __forceinline__ void load_v_frag(uint32_t v_base, int ks, int nt, uin
 
 // From the tiles in shared memory. PENDING_K / PENDING_V: copy groups that may still be in flight when the K tile,
 // then the V tile, are needed (those of later pages). Ends with the CTA in step.
-template <int HD, int PENDING_K, int PENDING_V>
+template <int HD, int VD, int PENDING_K, int PENDING_V>
 __device__ __forceinline__ void compute_page(const PageJob& job, const uint32_t (&qa)[HD / 16][4], const TcArgs& a,
                                              uint32_t k_base, uint32_t v_base, bf16* p_s, float (*red_m)[MAX_G], float (*red_l)[MAX_G],
                                              float* __restrict__ part_o, float* __restrict__ part_ml) {
-    compute_page_core<HD, SyncCta>(
+    compute_page_core<HD, VD, SyncCta>(
         job, qa, a,
         [&](int ks, uint32_t (&kb)[4]) { load_k_frag<HD, TileSwz<HD>>(k_base, ks, kb); },
-        [&](int ks, int nt, uint32_t (&vb)[4]) { load_v_frag<HD, TileSwz<HD>>(v_base, ks, nt, vb); },
+        [&](int ks, int nt, uint32_t (&vb)[4]) { load_v_frag<VD, TileSwz<VD>>(v_base, ks, nt, vb); },
         [&]() { cp_async_wait<PENDING_K>(); __syncthreads(); },       // K has landed (V may still be in flight)
         [&]() { cp_async_wait<PENDING_V>(); __syncthreads(); },       // V has landed
         p_s, red_m, red_l, part_o, part_ml);
@@ -367,19 +370,20 @@ __device__ __forceinline__ void compute_page(const PageJob& job, const uint32_t 
 // built and measured slower: 5.7 against 3.9 ms a step at batch 64; three CTAs an SM, and each turn of the loop
 // pays the chain of dependent reads that finds its next page.)
 template <int HD> __device__ __forceinline__ void merge_pages(const float* __restrict__, const float* __restrict__, bf16* __restrict__,
-                                                              size_t, int, int, int, float*, float*, float*);
+                                                              size_t, int, int, int, float*, float*, float*,
+                                                                       int null_key = 0, float out_scale = 1.f, int vdo = HD);
 
 // MERGE: the CTA that finishes a (sequence, kv head) last also merges its pages (a count per pair, zero before the
 // first launch and left zero by every launch), which saves the merge's launch; without it the merge is a launch
 // of its own with a CTA per head.
-template <int HD, bool MERGE>
+template <int HD, int VD, bool MERGE>
 __global__ void __launch_bounds__(WARPS * 32)
 attn_decode_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
                       const int* __restrict__ kv_len, PageTable pt, TcArgs a,
                       float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ status,
                       unsigned* __restrict__ counters, bf16* __restrict__ out, int ldo) {
     __shared__ __align__(128) unsigned char k_s[KEYS * HD * 2];     // reused by the merge for the pages' weights
-    __shared__ __align__(128) unsigned char v_s[KEYS * HD * 2];     // reused by the merge for its series
+    __shared__ __align__(128) unsigned char v_s[KEYS * VD * 2];     // reused by the merge for its series
     __shared__ __align__(16) bf16 p_s[MAX_G * KEYS];  // probabilities [head][key], rows of 8 chunks, swizzled
     __shared__ float red_m[WARPS][MAX_G], red_l[WARPS][MAX_G];
     __shared__ int last_flag;
@@ -390,12 +394,13 @@ attn_decode_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
         write_empty_partial(job, a, part_ml);
         if (!MERGE) return;
     } else {
-        issue_page_copies<HD>(job, k_cache, v_cache, a, smem_u32(k_s), smem_u32(v_s));
+        issue_page_copies<HD, VD>(job, k_cache, v_cache, a, smem_u32(k_s), smem_u32(v_s));
         uint32_t qa[HD / 16][4];
         load_q_fragments<HD>(job, q, a, qa);
-        compute_page<HD, 1, 0>(job, qa, a, smem_u32(k_s), smem_u32(v_s), p_s, red_m, red_l, part_o, part_ml);
+        compute_page<HD, VD, 1, 0>(job, qa, a, smem_u32(k_s), smem_u32(v_s), p_s, red_m, red_l, part_o, part_ml);
     }
-    if (MERGE) {
+    if constexpr (MERGE) {
+        static_assert(HD == VD, "the merging form has one head width");
         const int b = job.b, g = job.g, G = a.H / a.KV;
         __syncthreads();                              // the CTA's partial is written ...
         if (threadIdx.x == 0) {
@@ -421,7 +426,7 @@ attn_decode_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
 template <int HD>
 __device__ __forceinline__ void merge_pages(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                             bf16* __restrict__ out_row, size_t r0g, int G, int S, int n_vis,
-                                            float* w_s, float* acc_s, float* inv_s) {
+                                            float* w_s, float* acc_s, float* inv_s, int null_key, float out_scale, int vdo) {
     // (G may also be 1 with r0g and out_row pointing at one head: a head's arithmetic does not involve the others.)
     constexpr int LPR = HD / 4, NS = WARPS * 32 / LPR;
     constexpr int AHEAD = 8;                          // output rows a thread fetches before it has their weights
@@ -464,7 +469,9 @@ __device__ __forceinline__ void merge_pages(const float* __restrict__ part_o, co
             ls = fmaf(ml.y, w, ls);
         }
         ls = warp_sum(ls);
-        if (lane == 0) inv_s[i] = ls > 0.f ? 1.0f / ls : 0.f;
+        // the term without a key counts exp(0 - max); where that overflows, the keys' share of the softmax is zero
+        if (null_key && ls > 0.f) ls += expf(-mmax);
+        if (lane == 0) inv_s[i] = ls > 0.f ? out_scale / ls : 0.f;
     }
     __syncthreads();
     for (int i = 0; i < G; i++) {
@@ -487,11 +494,11 @@ __device__ __forceinline__ void merge_pages(const float* __restrict__ part_o, co
             add(__ldcg(reinterpret_cast<const float4*>(part_o + (r0h + s2) * HD) + ld4), w_s[i * S + s2]);
         reinterpret_cast<float4*>(acc_s + slot * HD)[ld4] = acc;
         __syncthreads();
-        for (int d = tid; d < HD; d += WARPS * 32) {
+        for (int d = tid; d < vdo; d += WARPS * 32) {
             float os = 0.f;
 #pragma unroll
             for (int k = 0; k < NS; k++) os += acc_s[k * HD + d];
-            out_row[(size_t)i * HD + d] = __float2bfloat16_rn(os * inv_s[i]);
+            out_row[(size_t)i * vdo + d] = __float2bfloat16_rn(os * inv_s[i]);
         }
         __syncthreads();
     }
@@ -501,7 +508,8 @@ __device__ __forceinline__ void merge_pages(const float* __restrict__ part_o, co
 template <int HD>
 __global__ void __launch_bounds__(WARPS * 32)
 attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out,
-                         const int* __restrict__ kv_len, int window, int keep_first, int H, int S, int ldo) {
+                         const int* __restrict__ kv_len, int window, int keep_first, int H, int S, int ldo,
+                         int null_key, float out_scale, int vdo) {
     constexpr int NS = WARPS * 32 / (HD / 4);
     extern __shared__ float w_s[];
     __shared__ __align__(16) float acc_s[NS * HD];
@@ -511,7 +519,8 @@ attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restri
     griddep_launch_small();
     const int hi = kv_len[b];
     const int n_vis = min(S, visible_pages(hi, window, keep_first).count());
-    merge_pages<HD>(part_o, part_ml, out + (size_t)b * ldo + (size_t)h * HD, ((size_t)b * H + h) * S, 1, S, n_vis, w_s, acc_s, inv_s);
+    merge_pages<HD>(part_o, part_ml, out + (size_t)b * ldo + (size_t)h * vdo, ((size_t)b * H + h) * S, 1, S, n_vis, w_s, acc_s, inv_s,
+                    null_key, out_scale, vdo);
 }
 
 // ---------------------------------------------------------------------------------------------------------
@@ -660,7 +669,7 @@ attn_decode_fused_kernel(const bf16* __restrict__ qkv, VecRef q_gain, VecRef k_g
         job.s = s; job.g = g; job.b = b; job.page = page;
         job.h_first = 1; job.h_last = 0; job.k_first = k_first; job.k_last = k_last; job.row0 = row0; job.empty = false;
         const TcArgs ta{a.H, a.KV, a.ldq, a.window, a.S, a.scale, 0, 1, 0.f};
-        compute_page<HD, 1, 0>(job, qa, ta, k_base, v_base, p_s, red_m, red_l, part_o, part_ml);
+        compute_page<HD, HD, 1, 0>(job, qa, ta, k_base, v_base, p_s, red_m, red_l, part_o, part_ml);
     }
 
     if (!MERGE) return;                               // the merge is a launch of its own (a CTA a head)
@@ -856,7 +865,7 @@ attn_decode_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
             __syncwarp();
             if (lane == 0) mbar_arrive(smem_u32(&bars[STAGES + st]));
             released = true;
-            compute_page_core<HD, SyncConsumers>(
+            compute_page_core<HD, HD, SyncConsumers>(
                 job, qa, a,
                 [&](int ks, uint32_t (&kb)[4]) { kb[0] = kf[ks][0]; kb[1] = kf[ks][1]; kb[2] = kf[ks][2]; kb[3] = kf[ks][3]; },
                 [&](int ks, int nt, uint32_t (&vb)[4]) { vb[0] = vf[ks][nt / 2][0]; vb[1] = vf[ks][nt / 2][1]; vb[2] = vf[ks][nt / 2][2]; vb[3] = vf[ks][nt / 2][3]; },
@@ -953,8 +962,8 @@ MYNAH_API int mynah_attn_decode_tc_capped(
     const void* q, void* out, int B, int H, int KV, int HD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window_in, int chunk, float scale, float softcap, int keep_first, int vdiv, int n_splits, float* scratch,
-    unsigned* counters, int* status, cudaStream_t stream);
+    int window_in, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, float out_scale, int vdo,
+    int n_splits, float* scratch, unsigned* counters, int* status, cudaStream_t stream);
 
 // The same with a chunk mask instead of the window (one of the two, 0: none) and a score scale given by the caller
 // (0: 1/sqrt(HD)).
@@ -964,40 +973,46 @@ MYNAH_API int mynah_attn_decode_tc_ex(
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
     int window_in, int chunk, float scale, int n_splits, float* scratch, unsigned* counters, int* status, cudaStream_t stream) {
     return mynah_attn_decode_tc_capped(q, out, B, H, KV, HD, ldq, ldo, k_cache, v_cache, kv_len, page_indptr, page_ids, page_base,
-                                       n_pages, window_in, chunk, scale, 0.f, 0, 1, n_splits, scratch, counters, status, stream);
+                                       n_pages, window_in, chunk, scale, 0.f, 0, 1, HD, 0, 1.0f, HD, n_splits, scratch, counters, status, stream);
 }
 
 // The same with capped scores (softcap c > 0: score <- c tanh(score / c), after the scale), first tokens that the window
 // keeps (keep_first, with a window and no chunk; the page lists must then hold every page of a sequence) and `vdiv` key
-// heads on one value head (the value cache is [n_pages, KV / vdiv, 64, HD]).
+// heads on one value head (the value cache is [n_pages, KV / vdiv, 64, VD]), value heads of a width VD of their own (64 or
+// 128; scratch of B * H * n_splits * (VD + 2) floats), one more softmax term of score 0 that has no value (null_key), a factor
+// on the output (out_scale) and output heads of `vdo` columns (at most VD: padding columns of the values are left out).
 MYNAH_API int mynah_attn_decode_tc_capped(
     const void* q, void* out, int B, int H, int KV, int HD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window_in, int chunk, float scale, float softcap, int keep_first, int vdiv, int n_splits, float* scratch,
-    unsigned* counters, int* status, cudaStream_t stream) {
+    int window_in, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, float out_scale, int vdo,
+    int n_splits, float* scratch, unsigned* counters, int* status, cudaStream_t stream) {
     if (B == 0) return 0;
     MYNAH_REQUIRE(window_in >= 0 && chunk >= 0 && !(window_in > 0 && chunk > 0), "attn_decode_tc: a window or a chunk, not both");
     MYNAH_REQUIRE(softcap >= 0.f && keep_first >= 0 && vdiv >= 1 && KV % vdiv == 0 && (keep_first == 0 || chunk == 0),
                   "attn_decode_tc: bad cap, kept tokens or value sharing");
+    MYNAH_REQUIRE((VD == 64 || VD == 128) && vdo > 0 && vdo <= VD, "attn_decode_tc: value heads of %d with %d output columns are not taken by this kernel", VD, vdo);
+    MYNAH_REQUIRE(counters == nullptr || (VD == HD && vdo == VD && !null_key && out_scale == 1.0f),
+                  "attn_decode_tc: the merging form takes plain heads of one width");
     const int window = chunk > 0 ? -chunk : window_in;
     MYNAH_REQUIRE(mynah_attn_decode_tc_supported(H, KV, HD), "attn_decode_tc: H=%d KV=%d head_dim=%d is not taken by this kernel", H, KV, HD);
     MYNAH_REQUIRE(ldq % 8 == 0, "attn_decode_tc: query row stride %d must be a multiple of 8", ldq);
     MYNAH_REQUIRE(n_splits >= 1 && n_splits <= 65535 && B <= 65535 && KV <= 65535, "attn_decode_tc: launch too large");
     MYNAH_REQUIRE(scratch != nullptr, "attn_decode_tc: no scratch memory given");
-    const TcArgs a{H, KV, ldq, window, n_splits, scale != 0.f ? scale : 1.0f / sqrtf((float)HD), window > 0 ? keep_first : 0, vdiv, softcap};
+    const TcArgs a{H, KV, ldq, window, n_splits, scale != 0.f ? scale : 1.0f / sqrtf((float)HD), window > 0 ? keep_first : 0, vdiv, softcap,
+                   null_key, out_scale, vdo};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     float* part_o = scratch;
-    float* part_ml = scratch + (size_t)B * H * n_splits * HD;
+    float* part_ml = scratch + (size_t)B * H * n_splits * VD;
     const dim3 grid(n_splits, KV, B);
     if (counters != nullptr) {
         MYNAH_REQUIRE((size_t)(H / KV) * n_splits * sizeof(float) <= MERGE_MAX_BYTES,
                       "attn_decode_tc: %d pages a sequence exceed what the merge holds", n_splits);
         if (HD == 128)
-            mynah_launch(attn_decode_tc_kernel<128, true>, grid, dim3(WARPS * 32), 0, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
+            mynah_launch(attn_decode_tc_kernel<128, 128, true>, grid, dim3(WARPS * 32), 0, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
                          kv_len, pt, a, part_o, part_ml, status, counters, (bf16*)out, ldo);
         else
-            mynah_launch(attn_decode_tc_kernel<64, true>, grid, dim3(WARPS * 32), 0, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
+            mynah_launch(attn_decode_tc_kernel<64, 64, true>, grid, dim3(WARPS * 32), 0, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
                          kv_len, pt, a, part_o, part_ml, status, counters, (bf16*)out, ldo);
         return mynah_check_launch("attn_decode_tc (merging)");
     }
@@ -1007,7 +1022,7 @@ MYNAH_API int mynah_attn_decode_tc_capped(
     const long long n_ctas = (long long)n_splits * KV * B;
     // (the stream form knows neither kept first tokens nor shared value heads: its jobs carry one range of rows a page and
     // one tensor map's coordinates for keys and values alike)
-    const bool as_stream = a.keep_first == 0 && a.vdiv == 1 && stream_mode() != 0 && B <= STREAM_MAX_SEQS && ((uintptr_t)q & 15) == 0 && ((uintptr_t)k_cache & 15) == 0 &&
+    const bool as_stream = a.keep_first == 0 && a.vdiv == 1 && VD == HD && stream_mode() != 0 && B <= STREAM_MAX_SEQS && ((uintptr_t)q & 15) == 0 && ((uintptr_t)k_cache & 15) == 0 &&
                            ((uintptr_t)v_cache & 15) == 0 && (stream_mode() == 2 || n_ctas >= (long long)mynah_sm_count() * 6 * 16);
     if (as_stream) {
         int rc;
@@ -1019,20 +1034,23 @@ MYNAH_API int mynah_attn_decode_tc_capped(
                                       : launch_stream<64, 2>(q, k_cache, v_cache, kv_len, pt, a, B, n_pages, part_o, part_ml, status, stream);
         if (rc) return rc;
     } else {
-        if (HD == 128)
-            mynah_launch(attn_decode_tc_kernel<128, false>, grid, dim3(WARPS * 32), 0, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
-                         kv_len, pt, a, part_o, part_ml, status, (unsigned*)nullptr, (bf16*)nullptr, 0);
-        else
-            mynah_launch(attn_decode_tc_kernel<64, false>, grid, dim3(WARPS * 32), 0, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
-                         kv_len, pt, a, part_o, part_ml, status, (unsigned*)nullptr, (bf16*)nullptr, 0);
+#define DTC_GO(HD_, VD_) mynah_launch(attn_decode_tc_kernel<HD_, VD_, false>, grid, dim3(WARPS * 32), 0, stream, (const bf16*)q, (const bf16*)k_cache, \
+                                      (const bf16*)v_cache, kv_len, pt, a, part_o, part_ml, status, (unsigned*)nullptr, (bf16*)nullptr, 0)
+        if (HD == 128 && VD == 128) DTC_GO(128, 128);
+        else if (HD == 128) DTC_GO(128, 64);
+        else if (VD == 128) DTC_GO(64, 128);
+        else DTC_GO(64, 64);
+#undef DTC_GO
         if (mynah_check_launch("attn_decode_tc")) return -1;
     }
     const size_t dyn = (size_t)n_splits * sizeof(float);
     MYNAH_REQUIRE(dyn <= MERGE_MAX_BYTES, "attn_decode_tc: %d pages a sequence exceed what the merge holds", n_splits);
-    if (HD == 128)
-        mynah_launch(attn_decode_merge_kernel<128>, dim3(H, B), dim3(WARPS * 32), dyn, stream, part_o, part_ml, (bf16*)out, kv_len, window, a.keep_first, H, n_splits, ldo);
+    if (VD == 128)
+        mynah_launch(attn_decode_merge_kernel<128>, dim3(H, B), dim3(WARPS * 32), dyn, stream, part_o, part_ml, (bf16*)out, kv_len, window, a.keep_first, H, n_splits, ldo,
+                     null_key, out_scale, vdo);
     else
-        mynah_launch(attn_decode_merge_kernel<64>, dim3(H, B), dim3(WARPS * 32), dyn, stream, part_o, part_ml, (bf16*)out, kv_len, window, a.keep_first, H, n_splits, ldo);
+        mynah_launch(attn_decode_merge_kernel<64>, dim3(H, B), dim3(WARPS * 32), dyn, stream, part_o, part_ml, (bf16*)out, kv_len, window, a.keep_first, H, n_splits, ldo,
+                     null_key, out_scale, vdo);
     return mynah_check_launch("attn_decode_merge");
 }
 
@@ -1074,9 +1092,9 @@ MYNAH_API int mynah_attn_decode_fused(
         if (mynah_check_launch("attn_decode_fused (pages)")) return -1;
         const size_t dyn_m = (size_t)n_splits * sizeof(float);
         if (HD == 128)
-            mynah_launch(attn_decode_merge_kernel<128>, dim3(H, B), dim3(WARPS * 32), dyn_m, stream, part_o, part_ml, (bf16*)out, kv_len, window, 0, H, n_splits, ldo);
+            mynah_launch(attn_decode_merge_kernel<128>, dim3(H, B), dim3(WARPS * 32), dyn_m, stream, part_o, part_ml, (bf16*)out, kv_len, window, 0, H, n_splits, ldo, 0, 1.0f, HD);
         else
-            mynah_launch(attn_decode_merge_kernel<64>, dim3(H, B), dim3(WARPS * 32), dyn_m, stream, part_o, part_ml, (bf16*)out, kv_len, window, 0, H, n_splits, ldo);
+            mynah_launch(attn_decode_merge_kernel<64>, dim3(H, B), dim3(WARPS * 32), dyn_m, stream, part_o, part_ml, (bf16*)out, kv_len, window, 0, H, n_splits, ldo, 0, 1.0f, HD);
         return mynah_check_launch("attn_decode_merge");
     }
     if (HD == 128)

@@ -51,6 +51,9 @@ struct PfArgs {
     int keep_first;                   // with a window: keys at positions below it are seen whatever their distance (every
                                       // page of the sequence must then be in the page list: nothing was given back)
     int vdiv;                         // kv head g reads value head g / vdiv (the value cache has KV / vdiv heads)
+    int null_key;                     // 1: the softmax has one more term, of score 0 and without a value
+    float out_scale;                  // factor on the output rows
+    int vdo;                          // columns of a head in the output rows (a multiple of 8, at most VD)
     float cap_in, cap_log2;           // capped scores (CAP kernels): c tanh(s scale / c) log2(e) = cap_log2 * tanh(s * cap_in)
     // The first key that the row at position p sees. Window and chunk both give a bound that does not fall as p
     // grows, so a tile's first row has the tile's lowest bound and its last row the highest.
@@ -126,14 +129,15 @@ __device__ __forceinline__ float capped_log2(float s, float cap_in, float cap_lo
     return s == -INFINITY ? -INFINITY : fmaf(t, cap_log2, -m);
 }
 
-template <int HD, int NS, bool CAP>
+template <int HD, int VD, int NS, bool CAP>
 __global__ void __launch_bounds__(THREADS, NS == 1 ? 2 : 1)
 attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* __restrict__ cu_q,
                             const int* __restrict__ kv_len, PageTable pt, PfArgs a, bf16* __restrict__ out,
                             int* __restrict__ status) {
-    constexpr int HALVES = HD / 64;
-    constexpr int TILE_BYTES = HALVES * HALF_BYTES;            // Q, K and V tiles: 128 rows x HD
+    constexpr int HALVES = HD / 64, VHALVES = VD / 64;
+    constexpr int TILE_BYTES = HALVES * HALF_BYTES;            // Q and K tiles: 128 rows x HD
+    constexpr int VTILE_BYTES = VHALVES * HALF_BYTES;          // V tiles: 128 rows x VD
     constexpr int PAGE_BYTES = PAGE_TOKENS * 128;              // one page in one half: 64 rows of 128 bytes
     constexpr int TMEM_COLS = NS == 2 ? 512 : 256;             // NS score buffers of 128 columns, the output behind them
     constexpr int O_COL = NS * 128;
@@ -144,7 +148,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     unsigned char* q_s = smem;
     unsigned char* k_s = q_s + TILE_BYTES;                     // NS stages
     unsigned char* v_s = k_s + NS * TILE_BYTES;                // NS stages
-    uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + NS * TILE_BYTES);
+    uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + NS * VTILE_BYTES);
     const uint32_t q_full = smem_u32(bars), k_full = smem_u32(bars + 1), v_full = smem_u32(bars + 3);   // [2] each, 8 bytes apart
     const uint32_t s_full = smem_u32(bars + 5), v_free = smem_u32(bars + 7);
     const uint32_t p_full = smem_u32(bars + 9), o_done = smem_u32(bars + 11), x_full = smem_u32(bars + 12);
@@ -225,13 +229,13 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     atomicOr(status, MYNAH_ST_PAGE_RANGE);
                     break;
                 }
-                const uint32_t bytes = ((p0 >= 0 ? 1 : 0) + (p1 >= 0 ? 1 : 0)) * HALVES * PAGE_BYTES;
+                const uint32_t n_pg = (p0 >= 0 ? 1 : 0) + (p1 >= 0 ? 1 : 0);
                 if (j >= NS && !mbar_wait(s_full + 8 * st, prev_use)) {     // the scores of tile j-NS are done: its K is free
                     atomicOr(status, MYNAH_ST_TIMEOUT);
                     break;
                 }
                 unsigned char* kd = k_s + st * TILE_BYTES;
-                mbar_expect_tx(k_full + 8 * st, bytes);
+                mbar_expect_tx(k_full + 8 * st, n_pg * HALVES * PAGE_BYTES);
 #pragma unroll
                 for (int hf = 0; hf < HALVES; hf++) {
                     if (p0 >= 0) tma_load_2d(smem_u32(kd + hf * HALF_BYTES), &map_k, hf * 64, (p0 * a.KV + kvh) * PAGE_TOKENS, k_full + 8 * st);
@@ -242,10 +246,10 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     atomicOr(status, MYNAH_ST_TIMEOUT);
                     break;
                 }
-                unsigned char* vd = v_s + st * TILE_BYTES;
-                mbar_expect_tx(v_full + 8 * st, bytes);
+                unsigned char* vd = v_s + st * VTILE_BYTES;
+                mbar_expect_tx(v_full + 8 * st, n_pg * VHALVES * PAGE_BYTES);
 #pragma unroll
-                for (int hf = 0; hf < HALVES; hf++) {
+                for (int hf = 0; hf < VHALVES; hf++) {
                     if (p0 >= 0) tma_load_2d(smem_u32(vd + hf * HALF_BYTES), &map_v, hf * 64, (p0 * KVV + kvh / a.vdiv) * PAGE_TOKENS, v_full + 8 * st);
                     if (p1 >= 0) tma_load_2d(smem_u32(vd + hf * HALF_BYTES + PAGE_BYTES), &map_v, hf * 64, (p1 * KVV + kvh / a.vdiv) * PAGE_TOKENS, v_full + 8 * st);
                 }
@@ -259,7 +263,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
     } else if (warp == 1) {
         if (lane == 0) {                                       // ---- MMA issuer
-            constexpr uint32_t idesc_s = idesc(BKV, false), idesc_o = idesc(HD, true);
+            constexpr uint32_t idesc_s = idesc(BKV, false), idesc_o = idesc(VD, true);
             const uint32_t t_o = tmem_base + O_COL;
             const uint32_t q_addr = smem_u32(q_s), k_addr = smem_u32(k_s), v_addr = smem_u32(v_s);
             auto scores = [&](int j) {                         // S[stage of j] = Q . K_j^T
@@ -294,7 +298,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 STAMP(j, 3);
 #pragma unroll
                 for (int k = 0; k < BKV / 16; k++)             // 16 keys a step: 8 columns of packed probabilities, 16 rows of V
-                    tc_mma_ts(t_o, tmem_base + st * BKV + (NS == 2 ? k * 8 : (k / 4) * 64 + (k % 4) * 8), desc_mn_major(v_addr + st * TILE_BYTES + k * 16 * 128, HALF_BYTES),
+                    tc_mma_ts(t_o, tmem_base + st * BKV + (NS == 2 ? k * 8 : (k / 4) * 64 + (k % 4) * 8), desc_mn_major(v_addr + st * VTILE_BYTES + k * 16 * 128, HALF_BYTES),
                               idesc_o, (j | k) != 0);
                 tc_commit(v_free + 8 * st);
                 tc_commit(o_done);
@@ -319,7 +323,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const bool bounded = a.bounded();
         const int lo_max = bounded ? a.row_lo(past + q0 + BQ - 1) : 0;    // the highest bound of any row of the tile
         const uint32_t t_row = tmem_base + ((uint32_t)(quad * 32) << 16);
-        const uint32_t t_o = t_row + O_COL + grp * (HD / 2);   // this thread's half of the row of O
+        const uint32_t t_o = t_row + O_COL + grp * (VD / 2);   // this thread's half of the row of O
         constexpr int HALF_KEYS = BKV / 2;
         float m_ref = -INFINITY, l = 0.f;                      // the maximum that the sums are scaled by; the sum over this thread's keys
         bool ok = true;
@@ -409,7 +413,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (!warp_wait(o_done, (j - 1) & 1)) { ok = false; break; }
                 tc_fence_after();
 #pragma unroll 1
-                for (int c = 0; c < HD / 64; c++) {
+                for (int c = 0; c < VD / 64; c++) {
                     uint32_t r[32];
                     tc_ld32(t_o + c * 32, r);
 #pragma unroll
@@ -472,8 +476,8 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (past_end || before_window) {
                 if (!warp_wait(v_full + 8 * st, use)) { ok = false; break; }
                 if ((past_end && row >= kvl - tile_key0) || (before_window && row < PAGE_TOKENS)) {
-                    for (int hf = grp; hf < HALVES; hf += 2) {
-                        uint4* dst = reinterpret_cast<uint4*>(v_s + st * TILE_BYTES + hf * HALF_BYTES + row * 128);
+                    for (int hf = grp; hf < VHALVES; hf += 2) {
+                        uint4* dst = reinterpret_cast<uint4*>(v_s + st * VTILE_BYTES + hf * HALF_BYTES + row * 128);
 #pragma unroll
                         for (int i = 0; i < 8; i++) dst[i] = make_uint4(0u, 0u, 0u, 0u);
                     }
@@ -497,16 +501,18 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (ok && !warp_wait(o_done, (n_tiles - 1) & 1)) ok = false;
         if (ok) {
             tc_fence_after();
-            const float inv = l > 0.f ? 1.0f / l : 0.f;
-            bf16* o_row = out + (size_t)(q_begin + q0 + row) * a.ldo + (size_t)h * HD + grp * (HD / 2);
+            // the term without a key counts 2^(0 - m); where that overflows, the keys' share of the softmax is zero
+            if (a.null_key && l > 0.f) l += ex2(-m_ref);
+            const float inv = l > 0.f ? a.out_scale / l : 0.f;
+            bf16* o_row = out + (size_t)(q_begin + q0 + row) * a.ldo + (size_t)h * a.vdo + grp * (VD / 2);
 #pragma unroll 1
-            for (int c = 0; c < HD / 64; c++) {
+            for (int c = 0; c < VD / 64; c++) {
                 uint32_t r[32];
                 tc_ld32(t_o + c * 32, r);
                 if (row < rows_valid) {
 #pragma unroll
                     for (int i = 0; i < 4; i++)
-                        reinterpret_cast<uint4*>(o_row + c * 32)[i] =
+                        if (grp * (VD / 2) + c * 32 + i * 8 < a.vdo) reinterpret_cast<uint4*>(o_row + c * 32)[i] =
                             make_uint4(pack2(__uint_as_float(r[8 * i]) * inv, __uint_as_float(r[8 * i + 1]) * inv),
                                        pack2(__uint_as_float(r[8 * i + 2]) * inv, __uint_as_float(r[8 * i + 3]) * inv),
                                        pack2(__uint_as_float(r[8 * i + 4]) * inv, __uint_as_float(r[8 * i + 5]) * inv),
@@ -528,11 +534,11 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #endif
 }
 
-template <int HD, int NS, bool CAP>
+template <int HD, int VD, int NS, bool CAP>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, int n_tokens, int B, int max_q_len, const int* cu_q,
            const int* kv_len, PageTable pt, PfArgs a, bf16* out, int* status, cudaStream_t stream) {
-    constexpr size_t smem = (1 + 2 * NS) * (size_t)(HD / 64) * HALF_BYTES + 128 + 2 * 2 * BQ * sizeof(float) + 1024;
-    auto kern = attn_prefill_tcgen05_kernel<HD, NS, CAP>;
+    constexpr size_t smem = ((1 + NS) * (size_t)(HD / 64) + NS * (size_t)(VD / 64)) * HALF_BYTES + 128 + 2 * 2 * BQ * sizeof(float) + 1024;
+    auto kern = attn_prefill_tcgen05_kernel<HD, VD, NS, CAP>;
     static bool opted = false;
     if (!opted) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -600,7 +606,8 @@ MYNAH_API int mynah_attn_prefill_tcgen05_capped(
     const void* q, void* out, int n_tokens, int B, int max_q_len, int H, int KV, int HD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* cu_q, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int* status, cudaStream_t stream);
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, float out_scale, int vdo,
+    int* status, cudaStream_t stream);
 
 // The same with a chunk mask beside the window (0: none) and a score scale given by the caller (0: 1/sqrt(HD)).
 MYNAH_API int mynah_attn_prefill_tcgen05_ex(
@@ -609,22 +616,27 @@ MYNAH_API int mynah_attn_prefill_tcgen05_ex(
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
     int window, int chunk, float scale, int* status, cudaStream_t stream) {
     return mynah_attn_prefill_tcgen05_capped(q, out, n_tokens, B, max_q_len, H, KV, HD, ldq, ldo, k_cache, v_cache, cu_q, kv_len,
-                                             page_indptr, page_ids, page_base, n_pages, window, chunk, scale, 0.f, 0, 1, status, stream);
+                                             page_indptr, page_ids, page_base, n_pages, window, chunk, scale, 0.f, 0, 1, HD, 0, 1.0f, HD, status, stream);
 }
 
 // The same with capped scores (softcap c > 0: score <- c tanh(score / c), after the scale), first tokens that the window
 // keeps (keep_first; the page lists must then hold every page of a sequence) and `vdiv` key heads on one value head (the
-// value cache is [n_pages, KV / vdiv, 64, HD]).
+// value cache is [n_pages, KV / vdiv, 64, VD]), value heads of a width VD of their own (64 or 128), one more softmax term of
+// score 0 that has no value (null_key), a factor on the output (out_scale) and output heads of `vdo` columns (a multiple of 8
+// up to VD: the padding columns of the values are left out).
 MYNAH_API int mynah_attn_prefill_tcgen05_capped(
     const void* q, void* out, int n_tokens, int B, int max_q_len, int H, int KV, int HD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* cu_q, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int* status, cudaStream_t stream) {
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, float out_scale, int vdo,
+    int* status, cudaStream_t stream) {
     if (B == 0 || max_q_len == 0 || n_tokens == 0) return 0;
     MYNAH_REQUIRE(window >= 0 && chunk >= 0, "attn_prefill_tcgen05: negative window or chunk");
     MYNAH_REQUIRE(softcap >= 0.f && keep_first >= 0 && vdiv >= 1 && KV % vdiv == 0 && (keep_first == 0 || chunk == 0),
                   "attn_prefill_tcgen05: bad cap, kept tokens or value sharing");
     MYNAH_REQUIRE(mynah_attn_prefill_tcgen05_supported(H, KV, HD), "attn_prefill_tcgen05: H=%d KV=%d head_dim=%d is not taken by this kernel", H, KV, HD);
+    MYNAH_REQUIRE((VD == 64 || VD == 128) && vdo > 0 && vdo <= VD && vdo % 8 == 0, "attn_prefill_tcgen05: value heads of %d with %d output columns are not taken by this kernel", VD, vdo);
+    MYNAH_REQUIRE(softcap == 0.f || VD == HD, "attn_prefill_tcgen05: capped scores need keys and values of one width");
     MYNAH_REQUIRE(ldq % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)out & 15) == 0 &&
                   ((uintptr_t)k_cache & 15) == 0 && ((uintptr_t)v_cache & 15) == 0,
                   "attn_prefill_tcgen05: rows must be 16-byte aligned (strides %d, %d)", ldq, ldo);
@@ -633,10 +645,10 @@ MYNAH_API int mynah_attn_prefill_tcgen05_capped(
     CUtensorMap mq, mk, mv;
     if (make_map(&mq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, n_tokens, (long long)H * HD, ldq, BQ, 64)) return -1;
     if (make_map(&mk, k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (long long)n_pages * KV * PAGE_TOKENS, HD, HD, PAGE_TOKENS, 64)) return -1;
-    if (make_map(&mv, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (long long)n_pages * (KV / vdiv) * PAGE_TOKENS, HD, HD, PAGE_TOKENS, 64)) return -1;
+    if (make_map(&mv, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (long long)n_pages * (KV / vdiv) * PAGE_TOKENS, VD, VD, PAGE_TOKENS, 64)) return -1;
     const float scale_used = scale != 0.f ? scale : 1.0f / sqrtf((float)HD);
     const PfArgs a{B, H, KV, ldo, window, scale_used * 1.4426950408889634f, chunk, keep_first, vdiv,
-                   softcap > 0.f ? scale_used / softcap : 0.f, softcap * 1.4426950408889634f};
+                   null_key, out_scale, vdo, softcap > 0.f ? scale_used / softcap : 0.f, softcap * 1.4426950408889634f};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     // Two CTAs an SM pay once there are several waves of CTAs (64 prompts of 2,048 tokens and 32 heads: 2.97 against
     // 3.34 ms; 4 prompts: 221 against 236 us); with one wave or two, the longest CTA's own chain sets the time and it
@@ -644,14 +656,20 @@ MYNAH_API int mynah_attn_prefill_tcgen05_capped(
     const int mode = stages_mode();
     const long long ctas = (long long)H * (ceil_div(n_tokens, BQ) + B);
     const int stages = mode != 0 ? mode : (ctas >= 8ll * mynah_sm_count() ? 1 : 2);
-#define PF_GO(HD_, NS_)                                                                                                         \
-    return softcap > 0.f ? launch<HD_, NS_, true>(mq, mk, mv, n_tokens, B, max_q_len, cu_q, kv_len, pt, a, (bf16*)out, status, stream) \
-                         : launch<HD_, NS_, false>(mq, mk, mv, n_tokens, B, max_q_len, cu_q, kv_len, pt, a, (bf16*)out, status, stream)
-    if (stages == 1) {
-        if (HD == 128) PF_GO(128, 1);
-        PF_GO(64, 1);
+#define PF_LAUNCH(HD_, VD_, NS_, CAP_) launch<HD_, VD_, NS_, CAP_>(mq, mk, mv, n_tokens, B, max_q_len, cu_q, kv_len, pt, a, (bf16*)out, status, stream)
+#define PF_GO(HD_, VD_) return stages == 1 ? PF_LAUNCH(HD_, VD_, 1, false) : PF_LAUNCH(HD_, VD_, 2, false)
+#define PF_GO_CAP(HD_) return stages == 1 ? PF_LAUNCH(HD_, HD_, 1, true) : PF_LAUNCH(HD_, HD_, 2, true)
+    if (softcap > 0.f) {
+        if (HD == 128) PF_GO_CAP(128);
+        PF_GO_CAP(64);
     }
-    if (HD == 128) PF_GO(128, 2);
-    PF_GO(64, 2);
+    if (HD == 128) {
+        if (VD == 128) PF_GO(128, 128);
+        PF_GO(128, 64);
+    }
+    if (VD == 128) PF_GO(64, 128);
+    PF_GO(64, 64);
+#undef PF_GO_CAP
+#undef PF_LAUNCH
 #undef PF_GO
 }

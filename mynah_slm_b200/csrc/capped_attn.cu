@@ -5,7 +5,9 @@
 //   capped_attn_prep   per token: every unit of `dim` values of the q and k projections (a head, or one map of a
 //                      head) gets its bias, an RMS norm with one gain shared by all units, and a rotation of its first
 //                      `rot` dimensions (pairs (i, i + rot/2) or (2i, 2i+1)); queries go to packed rows, keys and
-//                      (biased) values to the token's place in the paged cache. All of it in fp32.
+//                      (biased) values to the token's place in the paged cache. All of it in fp32. With a table of
+//                      query factors, q is multiplied by its position's factor at the end (a temperature that grows
+//                      with the position, say).
 //                      With M maps a head, query head h = g * R + j (R query heads a kv head) and map m go to
 //                      slot (g * M + m) * R + j of the packed row and key (g, m) to kv head g * M + m, so that the
 //                      attention kernels' own grouping (slot / R) pairs every query map with its key map, and kv
@@ -35,7 +37,8 @@ __global__ void __launch_bounds__(PREP_WARPS * 32)
 capped_attn_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* __restrict__ bias, VecRef q_gain,
                         VecRef k_gain, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                         const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, PageTable pt,
-                        T* __restrict__ k_cache, T* __restrict__ v_cache, CappedPrepArgs a, int* __restrict__ status) {
+                        T* __restrict__ k_cache, T* __restrict__ v_cache, const float* __restrict__ q_factor, CappedPrepArgs a,
+                        int* __restrict__ status) {
     __shared__ float unit[PREP_WARPS][32 * PREP_MAXC];
     griddep_launch_small();
     griddep_wait();
@@ -44,7 +47,7 @@ capped_attn_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const 
     if (b < 0) return;                                    // a padding row
     const int pos = tok_pos[t];
     const bool rotate = a.rot > 0 && cos_t != nullptr;
-    if (rotate && (pos < 0 || pos >= a.n_pos)) {
+    if ((rotate || q_factor != nullptr) && (pos < 0 || pos >= a.n_pos)) {
         if (threadIdx.x == 0) atomicOr(status, MYNAH_ST_POS_RANGE);
         return;
     }
@@ -101,6 +104,7 @@ capped_attn_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const 
     } else {
         dst = k_cache + (((size_t)page * a.Gk + (u - a.Hq)) * PAGE_TOKENS + pos % PAGE_TOKENS) * a.dimp;
     }
+    const float fq = is_q && q_factor != nullptr ? q_factor[pos] : 1.0f;
     for (int d = lane; d < a.dimp; d += 32) {
         float v = 0.f;
         if (d < a.dim) {
@@ -120,7 +124,7 @@ capped_attn_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const 
                 v = v * cr[i] + sign * mine[other] * sr[i];
             }
         }
-        dst[d] = from_f32<T>(v);
+        dst[d] = from_f32<T>(v * fq);
     }
 }
 
@@ -133,7 +137,8 @@ __global__ void __launch_bounds__(PREP_WARPS * 32)
 capped_attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* __restrict__ bias, VecRef q_gain,
                             VecRef k_gain, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                             const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, PageTable pt,
-                            T* __restrict__ k_cache, T* __restrict__ v_cache, CappedPrepArgs a, int* __restrict__ status) {
+                            T* __restrict__ k_cache, T* __restrict__ v_cache, const float* __restrict__ q_factor,
+                            CappedPrepArgs a, int* __restrict__ status) {
     griddep_launch_small();
     griddep_wait();
     const int t = blockIdx.x;
@@ -141,7 +146,7 @@ capped_attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, co
     if (b < 0) return;                                    // a padding row
     const int pos = tok_pos[t];
     const bool rotate = a.rot > 0 && cos_t != nullptr;
-    if (rotate && (pos < 0 || pos >= a.n_pos)) {
+    if ((rotate || q_factor != nullptr) && (pos < 0 || pos >= a.n_pos)) {
         if (threadIdx.x == 0) atomicOr(status, MYNAH_ST_POS_RANGE);
         return;
     }
@@ -232,6 +237,11 @@ capped_attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, co
     if (!on) return;
     T* dst;
     if (is_q) {
+        if (q_factor != nullptr) {
+            const float fq = q_factor[pos];
+#pragma unroll
+            for (int j = 0; j < 8; j++) v[j] *= fq;
+        }
         const int h = u / a.maps, m = u % a.maps;
         const int slot = ((h / a.R) * a.maps + m) * a.R + h % a.R;
         dst = q_out + (size_t)t * a.ldq + (size_t)slot * a.dim;
@@ -307,12 +317,14 @@ __global__ void head_gate_kernel(T* __restrict__ x, int ldx, const T* __restrict
 // and Gv heads of `vd` (v). bias: fp32 over those columns, or null. q_gain / k_gain: `dim` values each in gain_dtype,
 // or null for no norm. q_out: [T][ldq] packed queries of `dimp` values a slot; k_cache [pages][Gk][PAGE][dimp],
 // v_cache [pages][Gv][PAGE][vdp] (both null for a run that brings queries only). Padding columns are written as zeros.
+// q_factor: fp32 [n_pos], a factor on the query a position, or null; n_pos bounds it and the rotation's tables.
 MYNAH_API int mynah_capped_attn_prep(const void* qkv, int dtype, int T, int ld, void* q_out, int ldq, int Hq, int Gk, int Gv,
                                      int dim, int vd, int dimp, int vdp, int maps, int R, const float* bias,
                                      const void* q_gain, const void* k_gain, int gain_dtype, float eps, const float* cos_t,
                                      const float* sin_t, int rot, int interleaved, int n_pos, const int* tok_seq,
                                      const int* tok_pos, const int* page_indptr, const int* page_ids, const int* page_base,
-                                     int n_pages, void* k_cache, void* v_cache, int* status, cudaStream_t stream) {
+                                     int n_pages, void* k_cache, void* v_cache, const float* q_factor, int* status,
+                                     cudaStream_t stream) {
     if (T == 0) return 0;
     MYNAH_REQUIRE(T > 0 && Hq > 0 && Gk > 0 && Gv > 0 && dim > 0 && vd > 0 && maps > 0 && R > 0, "capped_attn_prep: bad sizes");
     MYNAH_REQUIRE(dim <= 32 * PREP_MAXC && dimp >= dim && vdp >= vd, "capped_attn_prep: a unit of %d values exceeds %d", dim, 32 * PREP_MAXC);
@@ -337,10 +349,10 @@ MYNAH_API int mynah_capped_attn_prep(const void* qkv, int dtype, int T, int ld, 
         const dim3 vgrid(T, ceil_div(n_qk, per_cta));
         if (dtype == MYNAH_F32)
             mynah_launch(capped_attn_prep_vec_kernel<float>, vgrid, dim3(PREP_WARPS * 32), 0, stream, (const float*)qkv, (float*)q_out, bias,
-                         qg, kg, cos_t, sin_t, tok_seq, tok_pos, pt, (float*)k_cache, (float*)v_cache, a, status);
+                         qg, kg, cos_t, sin_t, tok_seq, tok_pos, pt, (float*)k_cache, (float*)v_cache, q_factor, a, status);
         else if (dtype == MYNAH_BF16)
             mynah_launch(capped_attn_prep_vec_kernel<bf16>, vgrid, dim3(PREP_WARPS * 32), 0, stream, (const bf16*)qkv, (bf16*)q_out, bias,
-                         qg, kg, cos_t, sin_t, tok_seq, tok_pos, pt, (bf16*)k_cache, (bf16*)v_cache, a, status);
+                         qg, kg, cos_t, sin_t, tok_seq, tok_pos, pt, (bf16*)k_cache, (bf16*)v_cache, q_factor, a, status);
         else
             return mynah_fail("capped_attn_prep: unsupported dtype %d", dtype);
         return mynah_check_launch("capped_attn_prep");
@@ -350,10 +362,10 @@ MYNAH_API int mynah_capped_attn_prep(const void* qkv, int dtype, int T, int ld, 
     const dim3 grid(T, ceil_div(n_units, PREP_WARPS));
     if (dtype == MYNAH_F32)
         mynah_launch(capped_attn_prep_kernel<float>, grid, dim3(PREP_WARPS * 32), 0, stream, (const float*)qkv, (float*)q_out, bias,
-                     qg, kg, cos_t, sin_t, tok_seq, tok_pos, pt, (float*)k_cache, (float*)v_cache, a, status);
+                     qg, kg, cos_t, sin_t, tok_seq, tok_pos, pt, (float*)k_cache, (float*)v_cache, q_factor, a, status);
     else if (dtype == MYNAH_BF16)
         mynah_launch(capped_attn_prep_kernel<bf16>, grid, dim3(PREP_WARPS * 32), 0, stream, (const bf16*)qkv, (bf16*)q_out, bias, qg,
-                     kg, cos_t, sin_t, tok_seq, tok_pos, pt, (bf16*)k_cache, (bf16*)v_cache, a, status);
+                     kg, cos_t, sin_t, tok_seq, tok_pos, pt, (bf16*)k_cache, (bf16*)v_cache, q_factor, a, status);
     else
         return mynah_fail("capped_attn_prep: unsupported dtype %d", dtype);
     return mynah_check_launch("capped_attn_prep");

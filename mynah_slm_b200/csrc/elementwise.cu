@@ -413,6 +413,30 @@ __global__ void scale_f32_kernel(float* __restrict__ x, long long n, float s) {
     if (i < n) x[i] *= s;
 }
 
+// x[i] = c tanh(x[i] / c) in place (fp32): a head whose logits are capped.
+__global__ void softcap_f32_kernel(float* __restrict__ x, long long n, float c, float inv_c) {
+    griddep_launch_small();
+    griddep_wait();
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (i + 3 < n) {
+        float4 v = *reinterpret_cast<const float4*>(x + i);
+        v.x = c * tanhf(v.x * inv_c);
+        v.y = c * tanhf(v.y * inv_c);
+        v.z = c * tanhf(v.z * inv_c);
+        v.w = c * tanhf(v.w * inv_c);
+        *reinterpret_cast<float4*>(x + i) = v;
+    } else {
+        for (long long j = i; j < n; j++) x[j] = c * tanhf(x[j] * inv_c);
+    }
+}
+
+MYNAH_API int mynah_softcap_f32(float* x, long long n, float c, cudaStream_t stream) {
+    if (n == 0) return 0;
+    MYNAH_REQUIRE(n > 0 && c > 0.f && ((uintptr_t)x & 15) == 0, "softcap_f32: bad size %lld, cap or alignment", n);
+    mynah_launch(softcap_f32_kernel, dim3((unsigned)ceil_div_ll(ceil_div_ll(n, 4), 256)), dim3(256), 0, stream, x, n, c, 1.0f / c);
+    return mynah_check_launch("softcap_f32");
+}
+
 MYNAH_API int mynah_scale_f32(float* x, long long n, float s, cudaStream_t stream) {
     if (n == 0) return 0;
     MYNAH_REQUIRE(n > 0, "scale_f32: bad size %lld", n);

@@ -930,15 +930,15 @@ MYNAH_API int mynah_gemm_tcgen05(const void* A, const void* W, void* C, int M, i
 // Grouped product: W stacks `groups` matrices of group_rows rows each ([groups * group_rows, K]); the rows of A are sorted
 // by matrix and every matrix's rows padded to whole tiles of 128, and tile_group[m] (device, M / 128 entries) names the
 // matrix of row tile m. epilogue 1: C fp32 [M, N], N <= group_rows output columns of the tile's matrix; 5: the same with
-// the exact GELU on the rounded product, C bf16 [M, N]; 4: the clamped
-// gate, a matrix being N gate rows then N up rows (group_rows = 2 N), C bf16 [M, N]. M must be a multiple of 128.
+// the exact GELU on the rounded product, C bf16 [M, N]; 4: the clamped gate, 2: silu(gate) * up,
+// a matrix being N gate rows then N up rows (group_rows = 2 N), C bf16 [M, N]. M must be a multiple of 128.
 MYNAH_API int mynah_gemm_tcgen05_grouped(const void* A, const void* W, void* C, int M, int N, int K, int ldc, int epilogue,
                                          int groups, int group_rows, const int* tile_group, float gate_limit,
                                          float gate_alpha, int sm_count, int* status, cudaStream_t stream) {
     if (M == 0 || N == 0) return 0;
     MYNAH_REQUIRE(mynah_gemm_tcgen05_supported(M, N, K) && M % BM == 0, "gemm_tcgen05_grouped: M=%d N=%d K=%d is not taken", M, N, K);
-    MYNAH_REQUIRE((epilogue == EPI_F32 || epilogue == EPI_GATED || epilogue == EPI_GELU) && ldc >= N, "gemm_tcgen05_grouped: bad epilogue or output stride");
-    MYNAH_REQUIRE(groups > 0 && tile_group != nullptr && group_rows >= (epilogue == EPI_GATED ? 2 * N : N),
+    MYNAH_REQUIRE((epilogue == EPI_F32 || epilogue == EPI_GATED || epilogue == EPI_SWIGLU || epilogue == EPI_GELU) && ldc >= N, "gemm_tcgen05_grouped: bad epilogue or output stride");
+    MYNAH_REQUIRE(groups > 0 && tile_group != nullptr && group_rows >= (epi_glu(epilogue) ? 2 * N : N),
                   "gemm_tcgen05_grouped: the matrices do not hold the product's rows");
     const int csize = epilogue == EPI_F32 ? 4 : 2;
     MYNAH_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0 && ((uintptr_t)C & 15) == 0 && (ldc * csize) % 16 == 0,
@@ -955,6 +955,8 @@ MYNAH_API int mynah_gemm_tcgen05_grouped(const void* A, const void* W, void* C, 
     if (make_map(&mc, C, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, N, ldc, 32, 64)) return -1;
     if (epilogue == EPI_GELU)
         return launch_gemm<256, EPI_GELU, 1>(ma, mb, mc, M, N, K, 0, sm_count, status, stream, QkvEpilogue{}, tile_group, group_rows);
+    if (epilogue == EPI_SWIGLU)
+        return launch_gemm<256, EPI_SWIGLU, 1>(ma, mb, mc, M, N, K, N, sm_count, status, stream, QkvEpilogue{}, tile_group, group_rows);
     return launch_gemm<256, EPI_GATED, 1>(ma, mb, mc, M, N, K, N, sm_count, status, stream, QkvEpilogue{}, tile_group, group_rows,
                                           gate_limit, gate_alpha);
 }

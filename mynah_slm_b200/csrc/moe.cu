@@ -24,6 +24,11 @@
 //                 of neighbours, a group counts the sum of its two largest choice scores, only experts of the `keep`
 //                 best groups can be chosen (the lower index wins every tie); the `top` largest choice scores among
 //                 them are the token's experts, and each counts s (without the correction) times a constant.
+//                 Variants: scores softmax(W_r h) over all experts; a group counting its largest score; no correction.
+//                 A further row behind the router's matrix gives the gate of a shared expert: sigmoid of its product.
+//   shared expert   a feed-forward that every token passes: its rows, made by the ordinary products, join in moe_combine
+//                 times the token's gate
+//   clamped gate    with limit = infinity, alpha = 1 and shift 0 it is the plain silu(g) * u
 //
 // The grid of the two products covers the most tiles a step can have (pairs / rows-per-tile + experts); CTAs
 // beyond the step's tiles leave at once, so a captured step needs no count from the host.
@@ -91,7 +96,7 @@ enum MoeAct : int { MOE_ACT_CLAMPED_GATE = 0, MOE_ACT_GELU = 1 };
 
 struct MoeArgs {
     int top, D, F;
-    float limit, alpha;
+    float limit, alpha, shift;        // y = g sigmoid(alpha g) (u + shift), g and u clamped by limit
 };
 
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
@@ -134,7 +139,7 @@ moe_gate_up_kernel(const TA* __restrict__ h, const TA* __restrict__ w_gu, TA* __
             }
             const float gv = fminf(round_to<TA>(g[i][j]), a.limit);
             const float uv = fminf(fmaxf(round_to<TA>(u[i][j]), -a.limit), a.limit);
-            y[(size_t)p * a.F + c] = from_f32<TA>(gv * (1.0f / (1.0f + expf(-a.alpha * gv))) * (uv + 1.0f));
+            y[(size_t)p * a.F + c] = from_f32<TA>(gv * (1.0f / (1.0f + expf(-a.alpha * gv))) * (uv + a.shift));
         }
     }
 }
@@ -175,10 +180,12 @@ moe_down_kernel(const TA* __restrict__ y, const TA* __restrict__ w_down, float* 
 template <typename TA>
 __global__ void moe_combine_kernel(const float* __restrict__ o, const int* __restrict__ pair_expert,
                                    const int* __restrict__ row_of_pair, const float* __restrict__ pair_weight,
-                                   TA* __restrict__ out, int top, int D, float weight) {
+                                   TA* __restrict__ out, int top, int D, float weight, const float* __restrict__ shared,
+                                   const float* __restrict__ shared_gate) {
     griddep_launch_small();
     griddep_wait();
     const int t = blockIdx.x;
+    const float sg = shared != nullptr ? shared_gate[t] : 0.f;
     if (D % 4 == 0) {                                       // four columns a thread, 16-byte loads; a column's sum runs in the same order
         for (int c = threadIdx.x * 4; c < D; c += blockDim.x * 4) {
             float acc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -191,8 +198,18 @@ __global__ void moe_combine_kernel(const float* __restrict__ o, const int* __res
 #pragma unroll
                 for (int j = 0; j < 4; j++) acc[j] = pair_weight != nullptr ? fmaf(w, vv[j], acc[j]) : acc[j] + vv[j];
             }
+            float r[4];
 #pragma unroll
-            for (int j = 0; j < 4; j++) out[(size_t)t * D + c + j] = from_f32<TA>(pair_weight != nullptr ? acc[j] : acc[j] * weight);
+            for (int j = 0; j < 4; j++) r[j] = pair_weight != nullptr ? acc[j] : acc[j] * weight;
+            if (shared != nullptr) {
+                const float4 v = *reinterpret_cast<const float4*>(shared + (size_t)t * D + c);
+                r[0] = fmaf(sg, v.x, r[0]);
+                r[1] = fmaf(sg, v.y, r[1]);
+                r[2] = fmaf(sg, v.z, r[2]);
+                r[3] = fmaf(sg, v.w, r[3]);
+            }
+#pragma unroll
+            for (int j = 0; j < 4; j++) out[(size_t)t * D + c + j] = from_f32<TA>(r[j]);
         }
         return;
     }
@@ -204,7 +221,9 @@ __global__ void moe_combine_kernel(const float* __restrict__ o, const int* __res
             const float v = o[(size_t)(row_of_pair != nullptr ? row_of_pair[p] : p) * D + c];
             acc = pair_weight != nullptr ? fmaf(pair_weight[p], v, acc) : acc + v;
         }
-        out[(size_t)t * D + c] = from_f32<TA>(pair_weight != nullptr ? acc : acc * weight);
+        float r = pair_weight != nullptr ? acc : acc * weight;
+        if (shared != nullptr) r = fmaf(sg, shared[(size_t)t * D + c], r);
+        out[(size_t)t * D + c] = from_f32<TA>(r);
     }
 }
 
@@ -291,8 +310,8 @@ moe_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecRef bia
 template <typename TA>
 __global__ void __launch_bounds__(ROUTER_THREADS)
 moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecRef correction, const int* __restrict__ tok_seq,
-                        int* __restrict__ choice, float* __restrict__ pair_weight, int D, int E, int top, int groups, int keep,
-                        float weight_scale) {
+                        int* __restrict__ choice, float* __restrict__ pair_weight, float* __restrict__ shared_gate, int D, int E,
+                        int top, int groups, int keep, float weight_scale, int softmax_scores, int group_max) {
     __shared__ float sc[MOE_MAX_EXPERTS], ch[MOE_MAX_EXPERTS], gs[MOE_MAX_EXPERTS];
     griddep_wait();
     const int t = blockIdx.x;
@@ -301,12 +320,14 @@ moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecR
             choice[t * top + k] = -1;
             pair_weight[t * top + k] = 0.f;
         }
+        if (shared_gate != nullptr && threadIdx.x == 0) shared_gate[t] = 0.f;
         return;
     }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const TA* x = h + (size_t)t * D;
     const int D8 = D % 8 == 0 ? D : 0;
-    for (int e = warp; e < E; e += ROUTER_THREADS / 32) {
+    const int n_rows = shared_gate != nullptr ? E + 1 : E;           // the shared expert's gate is one more row
+    for (int e = warp; e < n_rows; e += ROUTER_THREADS / 32) {
         const TA* wr = w + (size_t)e * D;
         float acc = 0.f;
 #pragma unroll 2
@@ -320,13 +341,33 @@ moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecR
         for (int d = D8 + lane; d < D; d += 32) acc = fmaf(to_f32(x[d]), to_f32(wr[d]), acc);
         acc = warp_sum(acc);
         if (lane == 0) {
-            const float s = 1.0f / (1.0f + expf(-acc));
-            sc[e] = s;
-            ch[e] = s + correction.at(e);
+            if (e == E) {
+                shared_gate[t] = 1.0f / (1.0f + expf(-acc));
+            } else if (softmax_scores) {
+                sc[e] = acc;                                          // the logit, until all of them are there
+            } else {
+                const float s = 1.0f / (1.0f + expf(-acc));
+                sc[e] = s;
+                ch[e] = s + (correction.p != nullptr ? correction.at(e) : 0.f);
+            }
         }
     }
     __syncthreads();
     if (warp != 0) return;
+    if (softmax_scores) {
+        float zmax = -INFINITY, sum = 0.f;
+        for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, sc[e]);
+        zmax = warp_max(zmax);
+        for (int e = lane; e < E; e += 32) sum += expf(sc[e] - zmax);
+        const float inv = 1.0f / warp_sum(sum);
+        for (int e = lane; e < E; e += 32) {
+            const float z = sc[e], s = expf(z - zmax) * inv;
+            sc[e] = s;
+            // without a correction the choice goes by the logits, whose order the scores share (and which never round to equal zeros)
+            ch[e] = correction.p != nullptr ? s + correction.at(e) : z;
+        }
+        __syncwarp();
+    }
     if (keep < groups) {
         const int per = E / groups;
         for (int g = lane; g < groups; g += 32) {
@@ -336,7 +377,7 @@ moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecR
                 if (v > m1) { m2 = m1; m1 = v; }
                 else if (v > m2) m2 = v;
             }
-            gs[g] = per > 1 ? m1 + m2 : m1;
+            gs[g] = per > 1 && !group_max ? m1 + m2 : m1;
         }
         __syncwarp();
         // the best `keep` groups are marked by +inf in gs; the others' experts leave the choice
@@ -424,7 +465,7 @@ moe_gate_up_mma_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w_gu
                     }
                     const float gv = fminf(round_to<bf16>(acc[0][m][j][2 * half + q]), a.limit);
                     const float uv = fminf(fmaxf(round_to<bf16>(acc[NMAT - 1][m][j][2 * half + q]), -a.limit), a.limit);
-                    y[(size_t)p * a.F + c] = from_f32<bf16>(gv * (1.0f / (1.0f + expf(-a.alpha * gv))) * (uv + 1.0f));
+                    y[(size_t)p * a.F + c] = from_f32<bf16>(gv * (1.0f / (1.0f + expf(-a.alpha * gv))) * (uv + a.shift));
                 }
         }
 }
@@ -594,7 +635,8 @@ MYNAH_API int mynah_moe_max_tiles(int T, int top, int E) { return ceil_div(T * t
 static int moe_run(const void* h, int dtype, const int* tokens, const int* tok_seq, const int* table, const int* choice,
                    const float* pair_weight, const void* w_gu, const void* w_down, void* out, int out_f32, void* y, float* o,
                    int* ints, void* a_sorted, int T, int V, int top, int E, int D, int F, int act, float limit, float alpha,
-                   float weight, int* status, cudaStream_t stream) {
+                   float weight, int* status, cudaStream_t stream, float shift = 1.0f, const float* shared = nullptr,
+                   const float* shared_gate = nullptr) {
     const int P = T * top, BM = mynah_moe_tile_rows(T, top), max_tiles = mynah_moe_max_tiles(T, top, E);
     int* pair_expert = ints;
     int* perm = ints + P;
@@ -613,21 +655,22 @@ static int moe_run(const void* h, int dtype, const int* tokens, const int* tok_s
         if (act == MOE_ACT_GELU) {
             if (mynah_gemm_tcgen05_grouped(a_sorted, w_gu, y, m_pad, F, D, F, 5, E, F, tile_group, 0.f, 0.f, 0, status, stream) != 0) return -1;
         } else {
-            if (mynah_gemm_tcgen05_grouped(a_sorted, w_gu, y, m_pad, F, D, F, 4, E, 2 * F, tile_group, limit, alpha, 0, status, stream) != 0) return -1;
+            // shift 1: the clamped gate; shift 0 (then limit is infinite and alpha 1): the plain silu gate, an epilogue of its own
+            if (mynah_gemm_tcgen05_grouped(a_sorted, w_gu, y, m_pad, F, D, F, shift == 0.f ? 2 : 4, E, 2 * F, tile_group, limit, alpha, 0, status, stream) != 0) return -1;
         }
         if (mynah_gemm_tcgen05_grouped(y, w_down, o, m_pad, D, F, D, 1, E, D, tile_group, 0.f, 0.f, 0, status, stream) != 0) return -1;
         if (out_f32)
             mynah_launch(moe_combine_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)o, (const int*)pair_expert,
-                         (const int*)perm, pair_weight, (float*)out, top, D, weight);
+                         (const int*)perm, pair_weight, (float*)out, top, D, weight, shared, shared_gate);
         else
             mynah_launch(moe_combine_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const float*)o, (const int*)pair_expert,
-                         (const int*)perm, pair_weight, (bf16*)out, top, D, weight);
+                         (const int*)perm, pair_weight, (bf16*)out, top, D, weight, shared, shared_gate);
         return mynah_check_launch("moe_combine");
     }
     mynah_launch(moe_route_kernel, dim3(1), dim3(MOE_ROUTE_THREADS), 0, stream, tokens, tok_seq, table, choice, T, V, top, E, BM,
                  pair_expert, perm, tiles, max_tiles, status);
     if (mynah_check_launch("moe_route") != 0) return -1;
-    const MoeArgs a{top, D, F, limit, alpha};
+    const MoeArgs a{top, D, F, limit, alpha, shift};
     int rc;
     // bfloat16 rows that can move 16 bytes at a time take the tensor-core kernels
     const bool mma_ok = dtype == MYNAH_BF16 && D % 8 == 0 && F % 8 == 0 && !g_moe_plain &&
@@ -648,10 +691,10 @@ static int moe_run(const void* h, int dtype, const int* tokens, const int* tok_s
     if (rc != 0) return rc;
     if (dtype == MYNAH_F32 || out_f32)
         mynah_launch(moe_combine_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)o, (const int*)pair_expert,
-                     (const int*)nullptr, pair_weight, (float*)out, top, D, weight);
+                     (const int*)nullptr, pair_weight, (float*)out, top, D, weight, shared, shared_gate);
     else
         mynah_launch(moe_combine_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const float*)o, (const int*)pair_expert,
-                     (const int*)nullptr, pair_weight, (bf16*)out, top, D, weight);
+                     (const int*)nullptr, pair_weight, (bf16*)out, top, D, weight, shared, shared_gate);
     return mynah_check_launch("moe_combine");
 }
 
@@ -696,28 +739,34 @@ MYNAH_API int mynah_moe_router_ffn(const void* h, int dtype, const int* tok_seq,
 
 // The feed-forward with the group-limited scored router and the clamped-gate experts: scores sigmoid(W_r h) in fp32, the
 // choice by score + correction inside the `keep` best of `groups` equal groups of neighbouring experts, weights score *
-// weight_scale (not renormalised). w_router [E][D] in dtype, correction [E] in c_dtype; w_gu [E][2][F][D]; w_down [E][D][F];
+// weight_scale (not renormalised). softmax_scores: the scores are softmax(W_r h); group_max: a group counts its largest choice
+// score. The experts' gate: clamped (shift 1), or silu(g) u (shift 0, limit infinite, alpha 1). shared: fp32 rows [T][D] of a
+// shared expert, added times shared_gate [T], which the router writes from a further row of w_router ([E + 1][D]).
+// w_router [E][D] in dtype, correction [E] in c_dtype (or null); w_gu [E][2][F][D]; w_down [E][D][F];
 // out [T][D] in the activation type, or fp32 when out_f32. Scratch as for the learned router.
 MYNAH_API int mynah_moe_group_router_ffn(const void* h, int dtype, const int* tok_seq, const void* w_router, const void* correction,
                                          int c_dtype, const void* w_gu, const void* w_down, void* out, int out_f32, void* y, float* o,
                                          int* ints, void* a_sorted, int* choice, float* pair_weight, int T, int top, int E, int D,
-                                         int F, int groups, int keep, float weight_scale, float limit, float alpha, int* status,
+                                         int F, int groups, int keep, float weight_scale, int softmax_scores, int group_max, float limit,
+                                         float alpha, float shift, const float* shared, float* shared_gate, int* status,
                                          cudaStream_t stream) {
     if (T == 0) return 0;
     MYNAH_REQUIRE(T > 0 && top > 0 && E > 0 && top <= E && D > 0 && F > 0, "moe_group_router_ffn: bad sizes");
     MYNAH_REQUIRE(E <= MOE_MAX_EXPERTS, "moe_group_router_ffn: %d experts exceed %d", E, MOE_MAX_EXPERTS);
     MYNAH_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups, "moe_group_router_ffn: %d experts do not form %d groups of which %d are kept", E, groups, keep);
     MYNAH_REQUIRE(top <= keep * (E / groups), "moe_group_router_ffn: %d experts a token exceed those of %d kept groups", top, keep);
+    MYNAH_REQUIRE(shift == 1.0f || (shift == 0.f && limit > 3.0e38f && alpha == 1.0f), "moe_group_router_ffn: the experts' gate is the clamped one (shift 1) or the plain silu (shift 0, no limit, alpha 1)");
+    MYNAH_REQUIRE(shared == nullptr || shared_gate != nullptr, "moe_group_router_ffn: a shared expert's rows need its gates");
     const VecRef corr{correction, c_dtype};
     if (dtype == MYNAH_F32)
         mynah_launch(moe_group_router_kernel<float>, dim3(T), dim3(ROUTER_THREADS), 0, stream, (const float*)h, (const float*)w_router,
-                     corr, tok_seq, choice, pair_weight, D, E, top, groups, keep, weight_scale);
+                     corr, tok_seq, choice, pair_weight, shared_gate, D, E, top, groups, keep, weight_scale, softmax_scores, group_max);
     else if (dtype == MYNAH_BF16)
         mynah_launch(moe_group_router_kernel<bf16>, dim3(T), dim3(ROUTER_THREADS), 0, stream, (const bf16*)h, (const bf16*)w_router,
-                     corr, tok_seq, choice, pair_weight, D, E, top, groups, keep, weight_scale);
+                     corr, tok_seq, choice, pair_weight, shared_gate, D, E, top, groups, keep, weight_scale, softmax_scores, group_max);
     else
         return mynah_fail("moe_group_router_ffn: unsupported dtype %d", dtype);
     if (mynah_check_launch("moe_group_router") != 0) return -1;
     return moe_run(h, dtype, nullptr, tok_seq, nullptr, choice, pair_weight, w_gu, w_down, out, out_f32, y, o, ints, a_sorted, T, 1,
-                   top, E, D, F, MOE_ACT_CLAMPED_GATE, limit, alpha, 1.0f, status, stream);
+                   top, E, D, F, MOE_ACT_CLAMPED_GATE, limit, alpha, 1.0f, status, stream, shift, shared, shared_gate);
 }

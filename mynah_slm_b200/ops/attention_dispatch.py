@@ -110,32 +110,47 @@ def decode_masked(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: 
     kernels.attn_decode_general(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, chunk, scale, scratch)
 
 
+def _tc_capped_fits(HD: int, VD: int, scale: float, softcap: float, vdo: int) -> bool:
+    """Whether the tensor-core kernels take these heads: widths of 64 or 128 (one width for both under a cap), output heads
+    of whole 16-byte pieces."""
+    return USE_TC_MASKED and scale > 0.0 and VD in (64, 128) and (VD == HD or not softcap) and vdo % 8 == 0
+
+
 def prefill_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int, k_cache, v_cache, pages,
-                   window: int, scale: float, softcap: float, keep_first: int, vdiv: int) -> None:
-    """Prompt attention for mixers whose scores are capped, whose window keeps a sequence's first tokens, or whose
-    key heads share value heads (`vdiv` key heads a value head). Without any of the three it is `prefill_masked`; the
-    tcgen05 kernel takes bfloat16 heads of 64 or 128 with keys and values of one width, the general kernel the rest."""
-    if not softcap and not keep_first and vdiv == 1:
+                   window: int, scale: float, softcap: float, keep_first: int, vdiv: int, null_key: bool = False,
+                   out_scale: float = 1.0, vdo=None) -> None:
+    """Prompt attention for mixers whose scores are capped, whose window keeps a sequence's first tokens, whose key heads
+    share value heads (`vdiv` key heads a value head), whose softmax holds one more term of score 0 without a value
+    (`null_key`), whose output carries a factor, or whose output heads are narrower (`vdo` columns) than the stored value
+    heads. Without any of these it is `prefill_masked`; the tcgen05 kernel takes bfloat16 heads of 64 or 128, the general
+    kernel the rest."""
+    vdo = VD if vdo is None else int(vdo)
+    plain = not null_key and out_scale == 1.0 and vdo == VD
+    if plain and not softcap and not keep_first and vdiv == 1 and out.is_contiguous():
         prefill_masked(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, 0, scale)
         return
-    if (USE_TC_MASKED and USE_TCGEN05_PREFILL and HD == VD and scale > 0.0
+    if (USE_TCGEN05_PREFILL and _tc_capped_fits(HD, VD, scale, softcap, vdo)
             and kernels.attn_prefill_tcgen05_supported(q.dtype, H, KV, HD)):
         kernels.attn_prefill_tcgen05_capped(q, out, ctx, H, KV, HD, k_cache, v_cache, pages, window, scale, softcap,
-                                            keep_first, vdiv)
+                                            keep_first, vdiv, VD, null_key, out_scale, vdo)
         return
-    kernels.attn_prefill_capped(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, scale, softcap, keep_first, vdiv)
+    kernels.attn_prefill_capped(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, scale, softcap, keep_first, vdiv,
+                                null_key, out_scale, vdo)
 
 
 def decode_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int, k_cache, v_cache, pages,
-                  window: int, scale: float, softcap: float, keep_first: int, vdiv: int, scratch: torch.Tensor) -> None:
+                  window: int, scale: float, softcap: float, keep_first: int, vdiv: int, scratch: torch.Tensor,
+                  null_key: bool = False, out_scale: float = 1.0, vdo=None) -> None:
     """The same choice for a decode step."""
-    if not softcap and not keep_first and vdiv == 1:
+    vdo = VD if vdo is None else int(vdo)
+    plain = not null_key and out_scale == 1.0 and vdo == VD
+    if plain and not softcap and not keep_first and vdiv == 1 and out.is_contiguous():
         decode_masked(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, 0, scale, scratch)
         return
-    if (USE_TC_MASKED and HD == VD and scale > 0.0 and kernels.attn_decode_tc_supported(q.dtype, H, KV, HD)
+    if (_tc_capped_fits(HD, VD, scale, softcap, vdo) and kernels.attn_decode_tc_supported(q.dtype, H, KV, HD)
             and _tc_fits(H, KV, ctx.decode_splits)):
         kernels.attn_decode_tc_capped(q, out, ctx, H, KV, HD, k_cache, v_cache, pages, window, scale, softcap, keep_first,
-                                      vdiv, scratch)
+                                      vdiv, scratch, VD, null_key, out_scale, vdo)
         return
     kernels.attn_decode_capped(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, scale, softcap, keep_first, vdiv,
-                               scratch)
+                               scratch, null_key, out_scale, vdo)

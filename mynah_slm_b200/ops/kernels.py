@@ -825,6 +825,13 @@ def attn_decode_tc_masked(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: i
 
 
 # ------------------------------------------------------------------ latent attention, retention, routed experts
+def softcap_(x: torch.Tensor, c: float) -> torch.Tensor:
+    """x = c tanh(x / c) in place (fp32)."""
+    _chk(x, "rows", torch.float32)
+    call("mynah_softcap_f32", ptr(x), x.numel(), float(c), stream_ptr())
+    return x
+
+
 def scale_(x: torch.Tensor, s: float) -> torch.Tensor:
     """x *= s in place (fp32)."""
     _chk(x, "rows", torch.float32)
@@ -1199,9 +1206,11 @@ def sink_attn_tc(q: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor, k_ca
 def capped_attn_prep(qkv: torch.Tensor, q_out: torch.Tensor, Hq: int, Gk: int, Gv: int, dim: int, vd: int, dimp: int, vdp: int,
                      maps: int, R: int, bias: Optional[torch.Tensor], q_gain: Optional[torch.Tensor],
                      k_gain: Optional[torch.Tensor], eps: float, cos, sin, rot: int, interleaved: bool, ctx,
-                     pages: PageTableView, k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor]) -> None:
+                     pages: PageTableView, k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor],
+                     q_factor: Optional[torch.Tensor] = None) -> None:
     """Bias, per-unit RMS norm, rotation, packed queries and cache write of grouped-query attention with `maps`
-    score maps a head (csrc/capped_attn.cu). qkv: the projection's rows; q_out [T, Hq * dimp]."""
+    score maps a head (csrc/capped_attn.cu). qkv: the projection's rows; q_out [T, Hq * dimp]. q_factor: fp32 factors on
+    the query by position, or None."""
     _rows(qkv, "capped_attn_prep: projection")
     _chk(q_out, "packed queries", qkv.dtype, 2)
     writes = k_cache is not None
@@ -1225,30 +1234,44 @@ def capped_attn_prep(qkv: torch.Tensor, q_out: torch.Tensor, Hq: int, Gk: int, G
     n_pos = cos.shape[0] if cos is not None else 0
     if cos is not None and cos.shape[1] * 2 != rot:
         raise KernelError("capped_attn_prep: the rotation table does not match the rotated dims")
+    if q_factor is not None:
+        _chk(q_factor, "query factors", torch.float32, 1)
+        n_pos = min(n_pos, q_factor.numel()) if cos is not None else q_factor.numel()
     call("mynah_capped_attn_prep", ptr(qkv), code(qkv.dtype), qkv.shape[0], qkv.stride(0), ptr(q_out), q_out.shape[1], Hq, Gk, Gv,
          dim, vd, dimp, vdp, maps, R, ptr(bias), ptr(q_gain), ptr(k_gain), gd, float(eps), ptr(cos), ptr(sin),
          rot if cos is not None else 0, 1 if interleaved else 0, n_pos, ptr(ctx.tok_seq), ptr(ctx.tok_pos),
-         ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages, ptr(k_cache), ptr(v_cache), ptr(ctx.status),
-         stream_ptr())
+         ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages, ptr(k_cache), ptr(v_cache), ptr(q_factor),
+         ptr(ctx.status), stream_ptr())
+
+
+def _out_rows(out: torch.Tensor, q: torch.Tensor, H: int, width: int) -> None:
+    _rows(out, "attention output")
+    if out.dtype != q.dtype or out.shape[0] != q.shape[0] or out.shape[1] < H * width:
+        raise KernelError("attention output: the rows do not fit the heads")
 
 
 def attn_prefill_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int, k_cache, v_cache,
-                        pages: PageTableView, window: int, scale: float, softcap: float, keep_first: int, vdiv: int) -> None:
-    """The general prompt attention with capped scores, first tokens that the window keeps, and `vdiv` key heads on
-    one value head."""
+                        pages: PageTableView, window: int, scale: float, softcap: float, keep_first: int, vdiv: int,
+                        null_key: bool = False, out_scale: float = 1.0, vdo: Optional[int] = None) -> None:
+    """The general prompt attention with capped scores, first tokens that the window keeps, `vdiv` key heads on one value
+    head, one more softmax term of score 0 without a value (null_key), a factor on the output, and output heads of `vdo`
+    columns (None: VD). `out` may be a column slice of wider rows."""
     _chk(q, "q", dim=2)
-    _chk(out, "attention output", q.dtype, 2)
+    _out_rows(out, q, H, VD if vdo is None else vdo)
     call("mynah_attn_prefill_generic_capped", ptr(q), ptr(out), code(q.dtype), q.shape[0], ctx.B, ctx.max_q_len, H, KV, HD, VD,
-         q.shape[1], out.shape[1], ptr(k_cache), ptr(v_cache), ptr(ctx.cu_q), ptr(ctx.kv_len),
+         q.shape[1], out.stride(0), ptr(k_cache), ptr(v_cache), ptr(ctx.cu_q), ptr(ctx.kv_len),
          ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages, window or 0, 0, float(scale), float(softcap or 0.0),
-         int(keep_first or 0), int(vdiv), ptr(ctx.status), stream_ptr())
+         int(keep_first or 0), int(vdiv), 1 if null_key else 0, float(out_scale), int(vdo or 0), ptr(ctx.status), stream_ptr())
 
 
 def attn_prefill_tcgen05_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, k_cache: torch.Tensor,
                                 v_cache: torch.Tensor, pages: PageTableView, window: int, scale: float, softcap: float,
-                                keep_first: int, vdiv: int) -> None:
+                                keep_first: int, vdiv: int, VD: Optional[int] = None, null_key: bool = False,
+                                out_scale: float = 1.0, vdo: Optional[int] = None) -> None:
     """The tcgen05 prompt attention with capped scores, first tokens that the window keeps (the page lists must hold
-    every page: a cache that gives pages back does not go with kept tokens) and `vdiv` key heads on one value head."""
+    every page: a cache that gives pages back does not go with kept tokens) and `vdiv` key heads on one value head; value
+    heads of VD columns (64 or 128; None: HD), a null key, an output factor and output heads of `vdo` columns (a multiple
+    of 8) as in `attn_prefill_capped`."""
     for t, n in ((q, "q"), (out, "attention output")):
         _rows(t, "attn_prefill_tcgen05: " + n)
         if t.dtype != torch.bfloat16 or t.stride(0) % 8 or t.data_ptr() % 16:
@@ -1258,42 +1281,44 @@ def attn_prefill_tcgen05_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int,
     call("mynah_attn_prefill_tcgen05_capped", ptr(q), ptr(out), q.shape[0], ctx.B, ctx.max_q_len, H, KV, HD, q.stride(0),
          out.stride(0), ptr(k_cache), ptr(v_cache), ptr(ctx.cu_q), ptr(ctx.kv_len), ptr(pages.indptr), ptr(pages.ids),
          ptr(pages.base), pages.n_pages, window or 0, 0, float(scale), float(softcap or 0.0), int(keep_first or 0), int(vdiv),
-         ptr(ctx.status), stream_ptr())
+         int(VD or HD), 1 if null_key else 0, float(out_scale), int(vdo or VD or HD), ptr(ctx.status), stream_ptr())
 
 
 def attn_decode_tc_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, k_cache: torch.Tensor,
                           v_cache: torch.Tensor, pages: PageTableView, window: int, scale: float, softcap: float,
-                          keep_first: int, vdiv: int, scratch: torch.Tensor) -> None:
+                          keep_first: int, vdiv: int, scratch: torch.Tensor, VD: Optional[int] = None, null_key: bool = False,
+                          out_scale: float = 1.0, vdo: Optional[int] = None) -> None:
     """The tensor-core decode attention with capped scores, first tokens that the window keeps (the page lists must hold
-    every page) and `vdiv` key heads on one value head."""
+    every page) and `vdiv` key heads on one value head; the rest as in `attn_prefill_tcgen05_capped`."""
+    VD = int(VD or HD)
     for t, n in ((q, "q"), (out, "attention output")):
         _rows(t, "attn_decode_tc: " + n)
         if t.dtype != torch.bfloat16 or t.stride(0) % 8 or t.data_ptr() % 16:
             raise KernelError(f"attn_decode_tc: {n} must be bfloat16 rows, 16-byte aligned")
     _chk(scratch, "scratch", torch.float32)
-    need = ctx.B * H * ctx.decode_splits * (HD + 2)
+    need = ctx.B * H * ctx.decode_splits * (VD + 2)
     if scratch.numel() < need:
         raise KernelError(f"attn_decode_tc: scratch holds {scratch.numel()} floats, {need} are needed")
     call("mynah_attn_decode_tc_capped", ptr(q), ptr(out), ctx.B, H, KV, HD, q.stride(0), out.stride(0),
          ptr(k_cache), ptr(v_cache), ptr(ctx.kv_len), ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages,
-         window or 0, 0, float(scale), float(softcap or 0.0), int(keep_first or 0), int(vdiv), ctx.decode_splits,
-         ptr(scratch), None, ptr(ctx.status), stream_ptr())
+         window or 0, 0, float(scale), float(softcap or 0.0), int(keep_first or 0), int(vdiv), VD, 1 if null_key else 0,
+         float(out_scale), int(vdo or VD), ctx.decode_splits, ptr(scratch), None, ptr(ctx.status), stream_ptr())
     lib.add_launches(1)        # pages and their merge
 
 
 def attn_decode_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int, k_cache, v_cache,
                        pages: PageTableView, window: int, scale: float, softcap: float, keep_first: int, vdiv: int,
-                       scratch: torch.Tensor) -> None:
+                       scratch: torch.Tensor, null_key: bool = False, out_scale: float = 1.0, vdo: Optional[int] = None) -> None:
     _chk(q, "q", dim=2)
-    _chk(out, "attention output", q.dtype, 2)
+    _out_rows(out, q, H, VD if vdo is None else vdo)
     _chk(scratch, "scratch", torch.float32)
     need = ctx.B * H * ctx.decode_splits * (VD + 2)
     if scratch.numel() < need:
         raise KernelError(f"attn_decode: scratch holds {scratch.numel()} floats, {need} are needed")
-    call("mynah_attn_decode_capped", ptr(q), ptr(out), code(q.dtype), ctx.B, H, KV, HD, VD, q.shape[1], out.shape[1],
+    call("mynah_attn_decode_capped", ptr(q), ptr(out), code(q.dtype), ctx.B, H, KV, HD, VD, q.shape[1], out.stride(0),
          ptr(k_cache), ptr(v_cache), ptr(ctx.kv_len), ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages,
-         window or 0, 0, float(scale), float(softcap or 0.0), int(keep_first or 0), int(vdiv), ctx.decode_splits,
-         ptr(scratch), ptr(ctx.status), stream_ptr())
+         window or 0, 0, float(scale), float(softcap or 0.0), int(keep_first or 0), int(vdiv), 1 if null_key else 0,
+         float(out_scale), int(vdo or 0), ctx.decode_splits, ptr(scratch), ptr(ctx.status), stream_ptr())
     lib.add_launches(1)        # pages and their combination
 
 
@@ -1319,22 +1344,33 @@ def head_gate(x: torch.Tensor, gate: torch.Tensor, H: int, vd: int) -> torch.Ten
     return x
 
 
-def moe_group_router_ffn(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor, w_gu: torch.Tensor,
-                         w_down: torch.Tensor, ctx, top: int, groups: int, keep: int, weight_scale: float, limit: float,
-                         alpha: float) -> torch.Tensor:
+def moe_group_router_ffn(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], w_gu: torch.Tensor,
+                         w_down: torch.Tensor, ctx, top: int, groups: int, keep: int, weight_scale: float,
+                         limit: Optional[float], alpha: float, scores: str = "sigmoid", group_score: str = "top2",
+                         shared: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Experts picked by sigmoid scores (fp32) with a correction for the choice, inside the `keep` best of `groups` groups of
     neighbouring experts; clamped-gate experts; weights score * weight_scale (csrc/moe.cu). w_router [E, D], correction
-    [E], w_gu [E, 2, F, D], w_down [E, D, F]; returns [T, D] in the rows' type."""
+    [E] or None, w_gu [E, 2, F, D], w_down [E, D, F]; returns [T, D] in the rows' type. scores "softmax": over all
+    experts; group_score "max": a group counts its largest. limit None: the experts' gate is silu(g) * u. shared: fp32
+    rows [T, D] of a shared expert, added times sigmoid of the product with one more row of w_router ([E + 1, D])."""
     _chk(h, "rows", dim=2)
     _chk(w_router, "router weights", h.dtype, 2)
-    _chk(correction, "router correction", dim=1)
+    if correction is not None:
+        _chk(correction, "router correction", dim=1)
+    if scores not in ("sigmoid", "softmax") or group_score not in ("top2", "max"):
+        raise KernelError("moe_group_router_ffn: unknown scores or group score")
     _chk(w_gu, "gate/up weights", h.dtype, 4)
     _chk(w_down, "down weights", h.dtype, 3)
     T, D = h.shape
     E, _, F, _ = w_gu.shape
-    if (tuple(w_gu.shape) != (E, 2, F, D) or tuple(w_down.shape) != (E, D, F) or tuple(w_router.shape) != (E, D)
-            or correction.numel() != E or not 1 <= top <= E):
+    rows = E + (1 if shared is not None else 0)
+    if (tuple(w_gu.shape) != (E, 2, F, D) or tuple(w_down.shape) != (E, D, F) or tuple(w_router.shape) != (rows, D)
+            or (correction is not None and correction.numel() != E) or not 1 <= top <= E):
         raise KernelError("moe_group_router_ffn: sizes do not fit")
+    if shared is not None:
+        _chk(shared, "shared expert's rows", torch.float32, 2)
+        if shared.shape != h.shape:
+            raise KernelError("moe_group_router_ffn: the shared expert's rows do not fit")
     P_ = T * top
     dev = h.device
     grouped = int(lib.load().mynah_moe_grouped_rows(T, top, E, D, F, code(h.dtype)))
@@ -1345,11 +1381,66 @@ def moe_group_router_ffn(h: torch.Tensor, w_router: torch.Tensor, correction: to
     a = torch.empty((R, D), dtype=h.dtype, device=dev) if grouped else None
     ints = torch.empty((3 * P_ + 1 + 3 * int(lib.load().mynah_moe_max_tiles(T, top, E)) + R + R // 128 + 1,),
                        dtype=torch.int32, device=dev)
-    weights = torch.empty((P_,), dtype=torch.float32, device=dev)
+    weights = torch.empty((P_ + T,), dtype=torch.float32, device=dev)         # the pairs' weights, then the shared expert's gates
     choice = ints[ints.numel() - P_:]
+    plain = limit is None
     call("mynah_moe_group_router_ffn", ptr(h), code(h.dtype), ptr(ctx.tok_seq), ptr(w_router), ptr(correction),
-         code(correction.dtype), ptr(w_gu), ptr(w_down), ptr(out), 0, ptr(y), ptr(o), ptr(ints), ptr(a), ptr(choice),
-         ptr(weights), T, top, E, D, F, int(groups), int(keep), float(weight_scale), float(limit), float(alpha),
+         code(correction.dtype) if correction is not None else 0, ptr(w_gu), ptr(w_down), ptr(out), 0, ptr(y), ptr(o), ptr(ints),
+         ptr(a), ptr(choice), ptr(weights), T, top, E, D, F, int(groups), int(keep), float(weight_scale),
+         1 if scores == "softmax" else 0, 1 if group_score == "max" else 0, float("inf") if plain else float(limit),
+         1.0 if plain else float(alpha), 0.0 if plain else 1.0, ptr(shared), ptr(weights[P_:]) if shared is not None else None,
          ptr(ctx.status), stream_ptr())
     lib.add_launches(5 if grouped else 4)     # router, route, (gather,) two products, combine
+    return out
+
+
+# ------------------------------------------------------------------ linear attention with learned decays
+def gated_memory_chunk_min(n: int) -> int:
+    """From how many tokens in a step's longest piece a bfloat16 prompt runs chunk by chunk (`gated_memory`); 0: always token
+    by token. Returns the setting before; the two forms agree to rounding."""
+    return int(lib.load().mynah_gated_memory_chunk_min(int(n)))
+
+
+def gated_memory(kind: str, p: torch.Tensor, at: dict, w2: Optional[torch.Tensor], bias: torch.Tensor, w_norm: torch.Tensor,
+                 q_scale: float, state: dict, out: torch.Tensor, ctx, H: int, dim: int, vd: int, eps: float, tau: float = 1.0,
+                 cap: float = 1.0) -> torch.Tensor:
+    """A recurrence with its output norm and gate (csrc/gated_memory.cu). kind "gla": decays per key channel from the narrow
+    row at["a"] (w2 [H * dim, rank], bias [H * dim], tau); "mlstm": input and forget gates at["i"], at["f"] (bias [2 H], cap). p:
+    the projection's rows; at: first columns of q, k, v, g and those. state: "S" [slots + 1, H, dim, vd], for "mlstm" also
+    "n" and "m", fp32. out: rows (a column slice is fine) whose first H * vd columns are written."""
+    _rows(p, "gated_memory: projection")
+    _rows(out, "gated_memory: output")
+    gla = kind == "gla"
+    if not gla and kind != "mlstm":
+        raise KernelError(f"gated_memory: unknown kind {kind!r}")
+    S = state["S"]
+    _chk(S, "memory state", torch.float32, 4)
+    _chk(bias, "gate bias", torch.float32, 1)
+    _chk(w_norm, "norm weight", torch.float32, 1)
+    T = p.shape[0]
+    rank = 0
+    if gla:
+        _chk(w2, "decay matrix", p.dtype, 2)
+        rank = w2.shape[1]
+        if w2.shape[0] != H * dim or at["a"] + rank > p.shape[1]:
+            raise KernelError("gated_memory: the decay's matrix does not fit the heads")
+    else:
+        _chk(state["n"], "normaliser state", torch.float32, 3)
+        _chk(state["m"], "stabiliser state", torch.float32, 2)
+        if tuple(state["n"].shape[1:]) != (H, dim) or state["m"].shape[1] != H or max(at["i"], at["f"]) + H > p.shape[1]:
+            raise KernelError("gated_memory: the states or the gates do not fit the heads")
+    if (tuple(S.shape[1:]) != (H, dim, vd) or bias.numel() != (H * dim if gla else 2 * H) or w_norm.numel() != H * vd
+            or max(at["q"], at["k"]) + H * dim > p.shape[1] or max(at["v"], at["g"]) + H * vd > p.shape[1]
+            or out.dtype != p.dtype or out.shape[0] != T or out.shape[1] < H * vd):
+        raise KernelError("gated_memory: sizes do not fit")
+    q_len = 1 if ctx.is_decode else int(ctx.max_q_len)
+    need = int(lib.load().mynah_gated_memory_scratch_floats(0 if gla else 1, code(p.dtype), T, ctx.B, H, dim, vd, rank, q_len))
+    scratch = torch.empty((need,), dtype=torch.float32, device=p.device) if need else None
+    call("mynah_gated_memory", 0 if gla else 1, ptr(p), p.stride(0), at["q"], at["k"], at["v"], at["g"],
+         at["a"] if gla else at["i"], 0 if gla else at["f"], code(p.dtype), ptr(w2), rank, ptr(bias), ptr(w_norm), float(q_scale),
+         1.0 / float(tau), float(cap), float(eps), ptr(S), None if gla else ptr(state["n"]), None if gla else ptr(state["m"]),
+         S.shape[0] - 1, ptr(out), out.stride(0), 0, ptr(ctx.cu_q), ptr(ctx.slots), ctx.B, T, H, dim, vd, q_len, ptr(scratch),
+         stream_ptr())
+    if need:
+        lib.add_launches(2)
     return out

@@ -130,20 +130,25 @@ _SIGNATURES: dict[str, list] = {
                              c_float, P, P, P, P],
     "mynah_retention_scan": [P, P, P, c_int, c_int, c_int, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P],
     "mynah_attn_prefill_tcgen05_capped": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, P, P],
+                                          P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_float, c_int,
+                                          P, P],
     "mynah_attn_decode_tc_capped": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P, P, P, P, P, c_int,
-                                    c_int, c_int, c_float, c_float, c_int, c_int, c_int, P, P, P, P],
+                                    c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_float, c_int, c_int, P, P, P, P],
     "mynah_attn_prefill_generic_capped": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, P, P],
+                                          P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_float, c_int, P, P],
     "mynah_attn_decode_capped": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                 P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, P, P, P],
+                                 P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_float, c_int,
+                                 c_int, P, P, P],
     "mynah_capped_attn_prep": [P, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                               P, P, P, c_int, c_float, P, P, c_int, c_int, c_int, P, P, P, P, P, c_int, P, P, P, P],
+                               P, P, P, c_int, c_float, P, P, c_int, c_int, c_int, P, P, P, P, P, c_int, P, P, P, P, P],
     "mynah_diff_combine": [P, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, P, P],
     "mynah_head_gate": [P, c_int, c_int, c_int, P, c_int, c_int, c_int, P],
     "mynah_residual_add_row": [P, P, c_longlong, c_int, P],
     "mynah_moe_group_router_ffn": [P, c_int, P, P, P, c_int, P, P, P, c_int, P, P, P, P, P, P, c_int, c_int, c_int, c_int,
-                                   c_int, c_int, c_int, c_float, c_float, c_float, P, P],
+                                   c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_float, c_float, P, P, P, P],
+    "mynah_softcap_f32": [P, c_longlong, c_float, P],
+    "mynah_gated_memory": [c_int, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, c_int, P, P, c_float, c_float, c_float,
+                           c_float, P, P, P, c_int, P, c_int, c_int, P, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P],
     "mynah_moe_table_ffn": [P, c_int, P, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_float, c_float, c_float, P, P],
 }
@@ -189,11 +194,14 @@ def load() -> ctypes.CDLL:
     lib.mynah_gemm_tcgen05_splits_k.argtypes = [c_int, c_int, c_int, c_int]
     lib.mynah_gemv_decode_supported.restype = c_int
     lib.mynah_gemv_decode_supported.argtypes = [c_int, c_int, c_int]
-    for name in ("mynah_moe_plain", "mynah_retention_chunk_min", "mynah_head_linear_plain", "mynah_moe_grouped_min"):
+    for name in ("mynah_moe_plain", "mynah_retention_chunk_min", "mynah_head_linear_plain", "mynah_moe_grouped_min",
+                 "mynah_gated_memory_chunk_min"):
         getattr(lib, name).restype = c_int
         getattr(lib, name).argtypes = [c_int]
     lib.mynah_retention_scratch_floats.restype = c_longlong
     lib.mynah_retention_scratch_floats.argtypes = [c_int, c_int, c_int, c_int]
+    lib.mynah_gated_memory_scratch_floats.restype = c_longlong
+    lib.mynah_gated_memory_scratch_floats.argtypes = [c_int] * 9
     lib.mynah_moe_grouped_rows.restype = c_int
     lib.mynah_moe_grouped_rows.argtypes = [c_int, c_int, c_int, c_int, c_int, c_int]
     lib.mynah_moe_max_tiles.restype = c_int

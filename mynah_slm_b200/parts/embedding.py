@@ -3,7 +3,8 @@
 Embedding: x = E[token], no scaling by sqrt(hidden) (mynah-slm
 src/arch_qwen3.c:186); a design that multiplies its embedding by a constant
 gives `scale` (the product is fp32), and one that multiplies its logits by a
-constant gives the head `logit_scale`. Head: logits = Head . h in fp32, where Head is the
+constant gives the head `logit_scale`; one that caps its logits gives
+`logit_softcap` c: c tanh(logits / c). Head: logits = Head . h in fp32, where Head is the
 embedding matrix when the configuration ties them and `lm_head.weight`
 otherwise; the configuration decides, not the presence of the tensor
 (docs/qwen3-arch.md:91-113: the official checkpoint ships a duplicate
@@ -45,6 +46,7 @@ class LinearHead(Head):
         self.V, self.D = int(spec["vocab_size"]), int(spec["dim"])
         self.embedding = embedding
         self.logit_scale = float(spec.get("logit_scale", 1.0))
+        self.logit_softcap = float(spec.get("logit_softcap") or 0.0)
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self) -> list[TensorSpec]:
@@ -59,7 +61,9 @@ class LinearHead(Head):
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         logits = kernels.linear(h, self.weight, out_dtype=torch.float32)
-        return logits if self.logit_scale == 1.0 else kernels.scale_(logits, self.logit_scale)
+        if self.logit_scale != 1.0:
+            logits = kernels.scale_(logits, self.logit_scale)
+        return kernels.softcap_(logits, self.logit_softcap) if self.logit_softcap else logits
 
 
 register_embedding("token_embedding", TokenEmbedding)

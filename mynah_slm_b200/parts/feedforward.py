@@ -2,7 +2,9 @@
 
 x -> W_down . (silu(W_gate . x) * (W_up . x)), no bias (mynah-slm
 src/arch_qwen3.c:229-234, src/kernels.c:193-205). Parameters: hidden_size,
-intermediate_size, activation (only "silu" is built), prefix. Gate and up are
+intermediate_size, activation (only "silu" is built), and either prefix (the
+tensors are then <prefix>gate_proj.weight and so on) or the tensors' names gate,
+up and down. Gate and up are
 kept as one fused matrix [2 * intermediate, hidden], gate rows first, so a
 step is two products instead of three.
 """
@@ -24,22 +26,23 @@ class SwiGLUDense(FeedForward):
         super().__init__(spec)
         self.D = int(spec["hidden_size"])
         self.F = int(spec["intermediate_size"])
-        self.prefix = str(spec["prefix"])
+        if spec.get("prefix") is not None:
+            self.names = {k: f"{spec['prefix']}{k}_proj.weight" for k in ("gate", "up", "down")}
+        else:
+            self.names = {k: str(spec[k]) for k in ("gate", "up", "down")}
         act = spec.get("activation", "silu")
         if act != "silu":
             raise ConfigError(f"swiglu_dense: activation {act!r} is not supported (only 'silu')")
         self.w_gate_up = self.w_down = None
 
     def tensor_specs(self) -> list[TensorSpec]:
-        p = self.prefix
-        return [TensorSpec(p + "gate_proj.weight", (self.F, self.D)),
-                TensorSpec(p + "up_proj.weight", (self.F, self.D)),
-                TensorSpec(p + "down_proj.weight", (self.D, self.F))]
+        n = self.names
+        return [TensorSpec(n["gate"], (self.F, self.D)), TensorSpec(n["up"], (self.F, self.D)), TensorSpec(n["down"], (self.D, self.F))]
 
     def bind(self, tensors: Mapping[str, torch.Tensor], runtime) -> None:
-        p = self.prefix
-        self.w_gate_up = torch.cat([tensors[p + "gate_proj.weight"], tensors[p + "up_proj.weight"]], dim=0).contiguous()
-        self.w_down = tensors[p + "down_proj.weight"]
+        n = self.names
+        self.w_gate_up = torch.cat([tensors[n["gate"]], tensors[n["up"]]], dim=0).contiguous()
+        self.w_down = tensors[n["down"]]
 
     def streamed_tensors(self) -> list:
         return [self.w_gate_up, self.w_down]

@@ -35,8 +35,14 @@ tensors are `<expert_prefix><e>.up` and `.down`.
   the `top` largest choice scores among them; each counts s (without the correction) * weight_scale, not renormalised
   expert: the clamped-gate expert of `table_routed_experts` (limit, alpha)
 
+Variants, chosen by parameters: scores "softmax" (over all experts, instead of the sigmoid); group_score "max" (a group
+counts its largest choice score); correction None; limit None: the expert is W_down (silu(W_gate h) * (W_up h)). With
+`shared`, a feed-forward of that last form that every token passes (its intermediate size, and its tensors'
+`shared_prefix`), multiplied by sigmoid(w . h), one number a token (w: `shared_gate`), is added.
+
 Parameters: hidden_size, intermediate_size, experts, top, groups (1), keep (= groups), weight_scale (1), limit, alpha
-(1.702), router, correction (tensor names) and expert_prefix.
+(1.702), scores ("sigmoid"), group_score ("top2"), router, correction (tensor names), expert_prefix, and optionally
+shared, shared_prefix, shared_gate.
 """
 from __future__ import annotations
 
@@ -138,9 +144,16 @@ class GroupRouterExperts(FeedForward):
         self.groups = int(spec.get("groups", 1))
         self.keep = int(spec.get("keep", self.groups))
         self.weight_scale = float(spec.get("weight_scale", 1.0))
-        self.limit = float(spec["limit"])
+        self.limit = None if spec["limit"] is None else float(spec["limit"])
         self.alpha = float(spec.get("alpha", 1.702))
-        self.router_name, self.correction_name = str(spec["router"]), str(spec["correction"])
+        self.scores, self.group_score = str(spec.get("scores", "sigmoid")), str(spec.get("group_score", "top2"))
+        self.router_name = str(spec["router"])
+        self.correction_name = str(spec["correction"]) if spec.get("correction") is not None else None
+        self.FS = int(spec.get("shared") or 0)
+        self.shared_prefix = str(spec["shared_prefix"]) if self.FS else ""
+        self.shared_gate = str(spec["shared_gate"]) if self.FS else None
+        if self.scores not in ("sigmoid", "softmax") or self.group_score not in ("top2", "max"):
+            raise ConfigError(f"group_router_experts: scores {self.scores!r} or group score {self.group_score!r} is not built in")
         self.prefix = str(spec["expert_prefix"])
         if self.E > 1024:
             raise ConfigError(f"group_router_experts: {self.E} experts exceed the 1024 that the routing kernel counts")
@@ -154,8 +167,13 @@ class GroupRouterExperts(FeedForward):
         return f"{self.prefix}{e}.{which}"
 
     def tensor_specs(self) -> list[TensorSpec]:
-        specs = [TensorSpec(self.router_name, (self.E, self.D), std=0.3),
-                 TensorSpec(self.correction_name, (self.E,), role="gain", init="normal", std=0.1)]
+        specs = [TensorSpec(self.router_name, (self.E, self.D), std=0.3)]
+        if self.correction_name is not None:
+            specs.append(TensorSpec(self.correction_name, (self.E,), role="gain", init="normal", std=0.1))
+        if self.FS:
+            p = self.shared_prefix
+            specs += [TensorSpec(p + "gate", (self.FS, self.D)), TensorSpec(p + "up", (self.FS, self.D)),
+                      TensorSpec(p + "down", (self.D, self.FS)), TensorSpec(self.shared_gate, (1, self.D))]
         for e in range(self.E):
             specs += [TensorSpec(self._name(e, "gate"), (self.F, self.D)), TensorSpec(self._name(e, "up"), (self.F, self.D)),
                       TensorSpec(self._name(e, "down"), (self.D, self.F))]
@@ -163,17 +181,28 @@ class GroupRouterExperts(FeedForward):
 
     def bind(self, tensors: Mapping[str, torch.Tensor], runtime) -> None:
         self.w_router = tensors[self.router_name].contiguous()
-        self.correction = tensors[self.correction_name].contiguous()
+        self.correction = tensors[self.correction_name].contiguous() if self.correction_name is not None else None
+        self.w_shared = None
+        if self.FS:
+            p = self.shared_prefix
+            self.w_router = torch.cat([self.w_router, tensors[self.shared_gate]], dim=0).contiguous()
+            self.w_shared = torch.cat([tensors[p + "gate"], tensors[p + "up"]], dim=0).contiguous()
+            self.w_shared_down = tensors[p + "down"]
         self.w_gu = torch.stack([torch.stack([tensors[self._name(e, "gate")], tensors[self._name(e, "up")]])
                                  for e in range(self.E)]).contiguous()
         self.w_down = torch.stack([tensors[self._name(e, "down")] for e in range(self.E)]).contiguous()
 
     def streamed_tensors(self) -> list:
-        return [self.w_router]          # of the experts a step reads only those its tokens pick
+        # of the experts a step reads only those its tokens pick
+        return [self.w_router] + ([self.w_shared, self.w_shared_down] if self.FS else [])
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
+        shared = None
+        if self.FS:
+            shared = kernels.linear(kernels.linear_swiglu(h, self.w_shared), self.w_shared_down, out_dtype=torch.float32)
         return kernels.moe_group_router_ffn(h, self.w_router, self.correction, self.w_gu, self.w_down, ctx, self.top,
-                                            self.groups, self.keep, self.weight_scale, self.limit, self.alpha)
+                                            self.groups, self.keep, self.weight_scale, self.limit, self.alpha, self.scores,
+                                            self.group_score, shared)
 
 
 register_ffn("group_router_experts", GroupRouterExperts)

@@ -92,6 +92,8 @@ def _register_builtin() -> None:
     register_architecture(gupizen.ARCHITECTURE, gupizen.GupizenConfig.from_dict, replace=True)
     from .config import gomuzen
     register_architecture(gomuzen.ARCHITECTURE, gomuzen.GomuzenConfig.from_dict, replace=True)
+    from .config import buludra
+    register_architecture(buludra.ARCHITECTURE, buludra.BuludraConfig.from_dict, replace=True)
 
 
 _register_builtin()
