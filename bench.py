@@ -9,6 +9,7 @@ and 64.
     python bench.py --design nedupel      (the Nedupel design beside Supisun and Qwen3 at equal size, likewise)
     python bench.py --design gupizen      (the Gupizen design beside Supisun, Nedupel and Qwen3 at equal size, likewise)
     python bench.py --design gomuzen      (the Gomuzen design beside Nedupel, Supisun and Qwen3 at equal size, likewise)
+    python bench.py --design buludra      (the Buludra design beside Gupizen, Nedupel and Qwen3 at equal size, likewise)
 
 One JSON line on stdout. A step is one decode step of the batch.
   value     decoded tokens per second, timed on the device with CUDA events
@@ -388,6 +389,31 @@ def gomuzen_config(shape: str, layers: int) -> dict:
             "layers": [pattern[i % 4] for i in range(layers)]}
 
 
+# The Buludra design at layer sizes that resemble a real model's, beside Gupizen (the closest existing design: attention
+# with a sink beside a recurrent unit, a recurrence with a decay per channel, routed experts), Nedupel (retention, gated
+# experts) and Qwen3 at equal width, depth, heads and vocabulary. Its layers repeat (gated linear attention, parallel,
+# parallel, attention): the linear attention has the Qwen3 shape's heads with a state of head size x head size each, the
+# attentions keep those heads, the matrix memory has half as many heads with a state of half the head size x the head
+# size; feed-forwards alternate between dense and 16 experts in 4 groups (2 kept) of half the dense width of which a token
+# uses 2, beside a shared expert of the same size.
+def buludra_config(shape: str, layers: int) -> dict:
+    c = dict(QWEN3_0_6B)
+    c.update(SHAPES[shape])
+    D, H, G, HD, F = c["hidden_size"], c["num_attention_heads"], c["num_key_value_heads"], c["head_dim"], c["intermediate_size"]
+    dense = {"kind": "dense", "ff": F}
+    moe = {"kind": "moe", "expert": {"ff": F // 2}, "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 2}},
+           "shared": {"ff": F // 2}}
+    gla = {"type": "gla", "mixer": {"heads": H, "dim": HD, "vdim": HD, "tau": 16.0, "decay_rank": 16}}
+    par = {"type": "parallel", "mixer": {
+        "left": {"heads": H, "kv_heads": G, "dim": HD, "vdim": HD, "scale": HD ** -0.5, "rot": {"dims": HD, "base": 1e6}},
+        "right": {"heads": H // 2, "dim": HD // 2, "vdim": HD, "gate_cap": 15.0}, "left_scale": 1.2, "right_scale": 0.9}}
+    att = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": HD, "vdim": HD, "scale": HD ** -0.5,
+                                          "q_temp": {"coef": 0.1, "every": 1024}}}
+    pattern = [gla, par, par, att]
+    return {"architecture": "Buludra", "vocab": c["vocab_size"], "width": D, "max_positions": 8192, "norm": {"eps": 1e-6},
+            "logit_softcap": 15.0, "layers": [dict(pattern[i % 4], mlp=moe if i % 2 else dense) for i in range(layers)]}
+
+
 def run_design(args) -> int:
     """`--design NAME`: prefill of one 2,048-token prompt and decode steps at --batch behind 2,048-token prompts, for
     the design and for the existing models at equal size (`--model` runs one of them: for a launch list of that model alone)."""
@@ -416,6 +442,9 @@ def run_design(args) -> int:
             arms.insert(0, ("gomuzen", gomuzen_config(shape, layers)))
         if args.design == "gupizen":
             arms.insert(0, ("gupizen", gupizen_config(shape, layers)))
+        if args.design == "buludra":
+            arms = [("buludra", buludra_config(shape, layers)), ("gupizen", gupizen_config(shape, layers)),
+                    ("nedupel", nedupel_config(shape, layers)), ("qwen3", q)]
         for name, cfg in arms:
             if args.model and args.model != name:
                 continue
@@ -523,9 +552,9 @@ def main() -> int:
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="prompt length of the decode phases")
     ap.add_argument("--shape", default="0.6b", choices=sorted(SHAPES), help="layer sizes, for --only runs (the full line is always 0.6b)")
     ap.add_argument("--workload", default="", choices=["", "4b", "8b"], help="run one of the two larger workloads instead")
-    ap.add_argument("--design", default="", choices=["", "supisun", "nedupel", "gupizen", "gomuzen"],
+    ap.add_argument("--design", default="", choices=["", "supisun", "nedupel", "gupizen", "gomuzen", "buludra"],
                     help="measure this design beside Qwen3 at equal size instead (prefill and decode; a line of its own)")
-    ap.add_argument("--model", default="", choices=["", "supisun", "nedupel", "gupizen", "gomuzen", "qwen3"], help="with --design: only this one of the models")
+    ap.add_argument("--model", default="", choices=["", "supisun", "nedupel", "gupizen", "gomuzen", "buludra", "qwen3"], help="with --design: only this one of the models")
     args = ap.parse_args()
 
     if args.impl == "reference":
