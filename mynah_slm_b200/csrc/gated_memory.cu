@@ -21,7 +21,7 @@
 //   gm_chunk_scan    S before every chunk, elementwise in chunk order, in place over U; the sequence's state at the end
 //   gm_chunk_out     a chunk's outputs from the state before it and its own scores, then norm and gate
 //
-// With b_t the running sum of log decays inside the chunk: o_t = sum_{s<=t} <q_t e^{b_t}, k_s e^{-b_s}> v_s + (q_t e^{b_t}) S_0.
+// With b_t the running sum of log decays inside the chunk (kept as binary logarithms, so e^ is 2^ in the kernels): o_t = sum_{s<=t} <q_t e^{b_t}, k_s e^{-b_s}> v_s + (q_t e^{b_t}) S_0.
 // GLA scales q and k around half the chunk's total per channel (exponents stay within half the total), and where a chunk's
 // total exceeds GLA_RANGE forms every score channel by channel instead (all exponents then <= 0). MLSTM needs no scaling of q
 // and k: with g_s = i_s - F_s and M_t = max(m_0, max_{s<=t} g_s), m_t = F_t + M_t, a score counts e^{g_s - M_t} and the old
@@ -41,7 +41,8 @@ enum GmKind : int { GLA = 0, MLSTM = 1 };
 
 constexpr int GC = 64;                  // tokens of a chunk
 constexpr int G_THREADS = 256;
-constexpr float GLA_RANGE = 60.f;       // total of log decays (of one channel, over a chunk) up to which q and k are scaled
+constexpr float GLA_RANGE = 86.f;       // total of binary log decays (of one channel, over a chunk) up to which q and k are scaled
+constexpr float LOG2E = 1.4426950408889634f;
 constexpr float MLSTM_FLOOR = 1e-6f;
 
 struct GmArgs {
@@ -58,6 +59,13 @@ struct GmState {
 };
 
 __device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+// log2(sigmoid(z)): the logarithm of 1 + 2^-|.| from the hardware's log2 (absolute error about 2^-22), by its series where the
+// summand is small, so that decays next to one keep their relative accuracy
+__device__ __forceinline__ float log2_sigmoid(float z) {
+    const float y = z * LOG2E, e = exp2f(-fabsf(y));
+    const float s = e < 0.015625f ? e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 0.33333334f), -0.5f), 1.0f) * LOG2E : __log2f(1.0f + e);
+    return fminf(y, 0.f) - s;
+}
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 template <int KIND> __device__ __forceinline__ float gate_act(float z) { return KIND == GLA ? z * sigmoid_f(z) : sigmoid_f(z); }
 
@@ -121,6 +129,8 @@ gm_token_kernel(const T* __restrict__ p, const T* __restrict__ w2, const float* 
     }
     for (int t = q0; t < q1; t++) {
         const T* row = p + (size_t)t * a.ld;
+        // the first column's gate and weight are on their way while the token is worked on
+        const float z_first = tid < vd ? to_f32(row[a.g_off + h * vd + tid]) : 0.f, w_first = tid < vd ? w_norm[h * vd + tid] : 0.f;
         __syncthreads();                                       // the token before is done (and m, n, S are in place)
         for (int c = tid; c < dim; c += NT) {
             qs[c] = to_f32(row[a.q_off + h * dim + c]) * a.q_scale;
@@ -129,11 +139,27 @@ gm_token_kernel(const T* __restrict__ p, const T* __restrict__ w2, const float* 
         for (int c = tid; c < vd; c += NT) vs[c] = to_f32(row[a.v_off + h * vd + c]);
         if (KIND == GLA) {
             for (int c = tid; c < a.rank; c += NT) rs[c] = to_f32(row[a.a_off + c]);
+            // the thread's row of W_2, too (up to 16 values; the first token of a step brings it from memory)
+            const bool short_row = a.rank <= 16 && (a.rank * sizeof(T)) % 32 == 0;
+            float w_row[16], b_first = 0.f;
+            if (tid < dim) {
+                b_first = bias[h * dim + tid];
+                if (short_row) {
+                    const T* w = w2 + (size_t)(h * dim + tid) * a.rank;
+#pragma unroll
+                    for (int r = 0; r < 16; r += 8)
+                        if (r < a.rank) load8(w + r, *reinterpret_cast<float(*)[8]>(w_row + r));
+                }
+            }
             __syncthreads();
             for (int c = tid; c < dim; c += NT) {
                 const T* w = w2 + (size_t)(h * dim + c) * a.rank;
                 float z = 0.f;
-                if ((a.rank * sizeof(T)) % 32 == 0) {              // rows of whole 32-byte groups: 8 values a load
+                if (c == tid && short_row) {
+#pragma unroll
+                    for (int r = 0; r < 16; r++)
+                        if (r < a.rank) z = fmaf(w_row[r], rs[r], z);
+                } else if ((a.rank * sizeof(T)) % 32 == 0) {              // rows of whole 32-byte groups: 8 values a load
                     for (int r = 0; r < a.rank; r += 8) {
                         float wv[8];
                         load8(w + r, wv);
@@ -143,7 +169,7 @@ gm_token_kernel(const T* __restrict__ p, const T* __restrict__ w2, const float* 
                 } else {
                     for (int r = 0; r < a.rank; r++) z = fmaf(to_f32(w[r]), rs[r], z);
                 }
-                as[c] = expf(log_sigmoid_f(z + bias[h * dim + c]) * a.inv_tau);
+                as[c] = expf(log_sigmoid_f(z + (c == tid ? b_first : bias[h * dim + c])) * a.inv_tau);
             }
         } else if (tid == 0) {
             const float i = a.cap * tanhf((to_f32(row[a.a_off + h]) + bias[h]) / a.cap);
@@ -211,8 +237,8 @@ gm_token_kernel(const T* __restrict__ p, const T* __restrict__ w2, const float* 
         }
         const float r = 1.0f / sqrtf(block_sum(ss, red32) / (float)vd + a.eps);
         for (int c = tid; c < vd; c += NT) {
-            const float z = to_f32(row[a.g_off + h * vd + c]);
-            out[(size_t)t * a.ldo + a.o_off + h * vd + c] = from_f32<T>(os[c] * r * w_norm[h * vd + c] * gate_act<KIND>(z));
+            const float z = c == tid ? z_first : to_f32(row[a.g_off + h * vd + c]), w = c == tid ? w_first : w_norm[h * vd + c];
+            out[(size_t)t * a.ldo + a.o_off + h * vd + c] = from_f32<T>(os[c] * r * w * gate_act<KIND>(z));
         }
     }
     __syncthreads();
@@ -264,14 +290,38 @@ __device__ __forceinline__ uint32_t addr_bt(uint32_t base, int ld, int k0, int n
     return base + (uint32_t)(((k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * ld + n0 + (lane >> 4) * 8) * 2);
 }
 
-// rows [0, nt) of `cols` values (a multiple of 8) into a tile of GC rows; the rest of the tile, up to colsP columns, is zero
+// rows [0, nt) of `cols` values (a multiple of 8) into a tile of GC rows; the rest of the tile, up to colsP columns, is zero.
+// The copies are asynchronous, one group: cp_async_wait and a barrier before the tile is read.
 __device__ __forceinline__ void load_tile(bf16* dst, int ld, const bf16* __restrict__ src, size_t ld_src, int nt, int cols, int colsP) {
     const int ch = colsP / 8;
     for (int i = threadIdx.x; i < GC * ch; i += G_THREADS) {
         const int r = i / ch, c = (i % ch) * 8;
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (r < nt && c < cols) v = *reinterpret_cast<const uint4*>(src + (size_t)r * ld_src + c);
-        *reinterpret_cast<uint4*>(dst + r * ld + c) = v;
+        const bool in = r < nt && c < cols;
+        cp_async_16(smem_u32(dst + r * ld + c), in ? src + (size_t)r * ld_src + c : src, in);
+    }
+    cp_async_commit();
+}
+// four 8-value pieces of a thread, numbers i0, i0 + G_THREADS, ... of the tile's GC x (colsP / 8): loaded together
+struct Pieces { int t[4], c[4]; bool in[4], on[4]; };
+__device__ __forceinline__ Pieces pieces_of(int i0, int nt, int cols, int colsP) {
+    Pieces p;
+    const int ch = colsP / 8;
+#pragma unroll
+    for (int u = 0; u < 4; u++) {
+        const int i = i0 + u * G_THREADS;
+        p.t[u] = i / ch;
+        p.c[u] = (i % ch) * 8;
+        p.on[u] = i < GC * ch;
+        p.in[u] = p.on[u] && p.t[u] < nt && p.c[u] < cols;
+    }
+    return p;
+}
+__device__ __forceinline__ void widen8(const uint4& u, float (&v)[8]) {
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        v[2 * i] = __uint_as_float(w[i] << 16);
+        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
     }
 }
 
@@ -340,7 +390,27 @@ gm_chunk_state_kernel(const bf16* __restrict__ p, const bf16* __restrict__ w2, c
     bf16* r2 = r1 + GC * LR;                                   // GLA: [dimP][LR] W_2's rows of this head
     const bf16* prow = p + (size_t)t0 * a.ld;
     load_tile(vs, LV, prow + a.v_off + h * vd, a.ld, nt, vd, vdP);
+    uint4 k_raw[4];                                            // the thread's first pieces of k, on their way from here on
+    {
+        const Pieces pc = pieces_of(tid, nt, dim, dimP);
+#pragma unroll
+        for (int u = 0; u < 4; u++) k_raw[u] = pc.in[u] ? *reinterpret_cast<const uint4*>(prow + (size_t)pc.t[u] * a.ld + a.k_off + h * dim + pc.c[u]) : make_uint4(0u, 0u, 0u, 0u);
+    }
     if (KIND == GLA) {
+        if (a.rank % 8 == 0 && a.a_off % 8 == 0) {             // (w2 is 16-byte aligned)
+            const int ch = rankP / 8;
+            for (int i = tid; i < (GC + dimP) * ch; i += G_THREADS) {
+                const int r = i / ch, c = (i % ch) * 8;
+                uint4 v = make_uint4(0u, 0u, 0u, 0u);
+                if (r < GC) {
+                    if (r < nt && c < a.rank) v = *reinterpret_cast<const uint4*>(prow + (size_t)r * a.ld + a.a_off + c);
+                    *reinterpret_cast<uint4*>(r1 + r * LR + c) = v;
+                } else {
+                    if (r - GC < dim && c < a.rank) v = *reinterpret_cast<const uint4*>(w2 + (size_t)(h * dim + r - GC) * a.rank + c);
+                    *reinterpret_cast<uint4*>(r2 + (r - GC) * LR + c) = v;
+                }
+            }
+        } else
         for (int i = tid; i < (GC + dimP) * rankP; i += G_THREADS) {
             const int r = i / rankP, c = i % rankP;
             if (r < GC) r1[r * LR + c] = (r < nt && c < a.rank) ? prow[(size_t)r * a.ld + a.a_off + c] : __float2bfloat16_rn(0.f);
@@ -371,7 +441,7 @@ gm_chunk_state_kernel(const bf16* __restrict__ p, const bf16* __restrict__ w2, c
             float run = 0.f;
 #pragma unroll 4
             for (int t = s * 16; t < s * 16 + 16; t++) {
-                if (t < nt) run += log_sigmoid_f(zb[t * LZ + c] + bc) * a.inv_tau;
+                if (t < nt) run = fmaf(log2_sigmoid(zb[t * LZ + c] + bc), a.inv_tau, run);
                 zb[t * LZ + c] = run;
             }
             seg[s * dimP + c] = run;
@@ -400,25 +470,38 @@ gm_chunk_state_kernel(const bf16* __restrict__ p, const bf16* __restrict__ w2, c
             sc.scal[((size_t)flat * a.H + h) * 2 + 1] = zb[nt - 1] + G;
         }
     }
-    for (int i = tid; i < GC * (dimP / 8); i += G_THREADS) {
-        const int t = i / (dimP / 8), c = (i % (dimP / 8)) * 8;
-        float kv[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        if (t < nt && c < dim) {
-            load8(prow + (size_t)t * a.ld + a.k_off + h * dim + c, kv);
-            if (KIND == GLA) {
+    for (int i0 = tid; i0 < GC * (dimP / 8); i0 += 4 * G_THREADS) {
+        const Pieces pc = pieces_of(i0, nt, dim, dimP);
+        if (i0 != tid) {
 #pragma unroll
-                for (int j = 0; j < 8; j++) kv[j] *= expf(zb[(nt - 1) * LZ + c + j] - zb[t * LZ + c + j]);
-            } else {
-                const float w = expf(zb[GC + t] - G);
-#pragma unroll
-                for (int j = 0; j < 8; j++) kv[j] *= w;
-            }
+            for (int u = 0; u < 4; u++) k_raw[u] = pc.in[u] ? *reinterpret_cast<const uint4*>(prow + (size_t)pc.t[u] * a.ld + a.k_off + h * dim + pc.c[u]) : make_uint4(0u, 0u, 0u, 0u);
         }
-        uint4 hi, lo;
-        split8(kv, hi, lo);
-        *reinterpret_cast<uint4*>(kh + t * LK + c) = hi;
-        *reinterpret_cast<uint4*>(kl + t * LK + c) = lo;
+#pragma unroll
+        for (int u = 0; u < 4; u++) {
+            if (!pc.on[u]) continue;
+            const int t = pc.t[u], c = pc.c[u];
+            float kv[8];
+            widen8(k_raw[u], kv);
+            if (pc.in[u]) {
+                if (KIND == GLA) {
+                    float be[8], bt[8];
+                    load8(zb + (nt - 1) * LZ + c, be);
+                    load8(zb + t * LZ + c, bt);
+#pragma unroll
+                    for (int j = 0; j < 8; j++) kv[j] *= exp2f(be[j] - bt[j]);
+                } else {
+                    const float w = expf(zb[GC + t] - G);
+#pragma unroll
+                    for (int j = 0; j < 8; j++) kv[j] *= w;
+                }
+            }
+            uint4 hi, lo;
+            split8(kv, hi, lo);
+            *reinterpret_cast<uint4*>(kh + t * LK + c) = hi;
+            *reinterpret_cast<uint4*>(kl + t * LK + c) = lo;
+        }
     }
+    cp_async_wait<0>();
     __syncthreads();
     const size_t fh = (size_t)flat * a.H + h;
     if (KIND == MLSTM) {
@@ -516,7 +599,7 @@ gm_chunk_scan_kernel(GmState st, GmScratch sc, const int* __restrict__ cu_q, con
             *u_of(c) = S;                                      // the state before the chunk
             float keep, add = 1.f;
             if (KIND == GLA) {
-                keep = expf(d[i].x);
+                keep = exp2f(d[i].x);
             } else {
                 if (e == 0) sc.m0[(size_t)(base + nch - 1 - c) * a.H + h] = m;
                 const float m_new = fmaxf(m + d[i].x, d[i].y);
@@ -563,9 +646,25 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
     bf16* As = ks;                                             // [2][GC][LA]
     const bf16* prow = p + (size_t)t0 * a.ld;
     const size_t fh = (size_t)flat * a.H + h;
-    load_tile(vs, LV, prow + a.v_off + h * vd, a.ld, nt, vd, vdP);
     float m0 = 0.f;
+    uint4 q_raw[4], k_raw[4];
+    float4 b_raw[4][2];
+    auto fetch_qkb = [&](const Pieces& pc) {
+#pragma unroll
+        for (int u = 0; u < 4; u++) {
+            q_raw[u] = k_raw[u] = make_uint4(0u, 0u, 0u, 0u);
+            b_raw[u][0] = b_raw[u][1] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (pc.in[u]) {
+                q_raw[u] = *reinterpret_cast<const uint4*>(prow + (size_t)pc.t[u] * a.ld + a.q_off + h * dim + pc.c[u]);
+                k_raw[u] = *reinterpret_cast<const uint4*>(prow + (size_t)pc.t[u] * a.ld + a.k_off + h * dim + pc.c[u]);
+                const float4* bp = reinterpret_cast<const float4*>(sc.b + ((size_t)(t0 + pc.t[u]) * a.H + h) * dim + pc.c[u]);
+                b_raw[u][0] = bp[0];
+                b_raw[u][1] = bp[1];
+            }
+        }
+    };
     if (KIND == GLA) {
+        fetch_qkb(pieces_of(tid, nt, dim, dimP));
         if (tid == 0) wide_s = 0;
         __syncthreads();
         const float* blast = sc.b + ((size_t)(t0 + nt - 1) * a.H + h) * dim;
@@ -576,43 +675,50 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
         }
         __syncthreads();
         const bool wide = wide_s != 0;
-        for (int i = tid; i < GC * (dimP / 8); i += G_THREADS) {
-            const int t = i / (dimP / 8), c = (i % (dimP / 8)) * 8;
-            float qv[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, kv[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-            if (t < nt && c < dim) {
-                float bv[8];
-                load8(prow + (size_t)t * a.ld + a.q_off + h * dim + c, qv);
-                load8(prow + (size_t)t * a.ld + a.k_off + h * dim + c, kv);
-                load8(sc.b + ((size_t)(t0 + t) * a.H + h) * dim + c, bv);
+        for (int i0 = tid; i0 < GC * (dimP / 8); i0 += 4 * G_THREADS) {
+            const Pieces pc = pieces_of(i0, nt, dim, dimP);
+            if (i0 != tid) fetch_qkb(pc);
+#pragma unroll
+            for (int u = 0; u < 4; u++) {
+                if (!pc.on[u]) continue;
+                const int t = pc.t[u], c = pc.c[u];
+                float qv[8], kv[8], ref[8];
+                widen8(q_raw[u], qv);
+                widen8(k_raw[u], kv);
+                const float bv[8] = {b_raw[u][0].x, b_raw[u][0].y, b_raw[u][0].z, b_raw[u][0].w, b_raw[u][1].x, b_raw[u][1].y, b_raw[u][1].z, b_raw[u][1].w};
+                load8(rf + c, ref);
 #pragma unroll
                 for (int j = 0; j < 8; j++) {
-                    const float ref = wide ? 0.f : rf[c + j];
-                    qv[j] *= a.q_scale * expf(bv[j] - ref);
-                    if (!wide) kv[j] *= expf(ref - bv[j]);
+                    const float x = wide ? bv[j] : bv[j] - ref[j];
+                    qv[j] *= a.q_scale * exp2f(x);
+                    if (!wide) kv[j] *= exp2f(-x);
+                }
+                uint4 hi, lo;
+                split8(qv, hi, lo);
+                *reinterpret_cast<uint4*>(qs + t * LK + c) = hi;
+                *reinterpret_cast<uint4*>(qs + GC * LK + t * LK + c) = lo;
+                if (!wide) {
+                    split8(kv, hi, lo);
+                    *reinterpret_cast<uint4*>(ks + t * LK + c) = hi;
+                    *reinterpret_cast<uint4*>(ks + GC * LK + t * LK + c) = lo;
                 }
             }
-            uint4 hi, lo;
-            split8(qv, hi, lo);
-            *reinterpret_cast<uint4*>(qs + t * LK + c) = hi;
-            *reinterpret_cast<uint4*>(qs + GC * LK + t * LK + c) = lo;
-            if (!wide) {
-                split8(kv, hi, lo);
-                *reinterpret_cast<uint4*>(ks + t * LK + c) = hi;
-                *reinterpret_cast<uint4*>(ks + GC * LK + t * LK + c) = lo;
-            }
         }
+        load_tile(vs, LV, prow + a.v_off + h * vd, a.ld, nt, vd, vdP);          // under the scores
     } else {
         load_tile(qs, LK, prow + a.q_off + h * dim, a.ld, nt, dim, dimP);
         load_tile(ks, LK, prow + a.k_off + h * dim, a.ld, nt, dim, dimP);
+        load_tile(vs, LV, prow + a.v_off + h * vd, a.ld, nt, vd, vdP);
         m0 = sc.m0[fh];
         mlstm_gates(p, bias, t0, nt, h, a, Fs, gs, Ms);
         for (int c = tid; c < dimP; c += G_THREADS) rf[c] = c < dim ? sc.un[fh * dim + c] : 0.f;
+        cp_async_wait<1>();                                    // q and k (the values land under the scores)
     }
     __syncthreads();
     const bool wide = KIND == GLA && wide_s != 0;
     if (KIND == MLSTM && tid < GC) Ms[tid] = fmaxf(Ms[tid], m0);       // (read by others behind the next barrier)
     if (KIND == GLA)                                                   // from here on the factor itself, for the state's rows
-        for (int c = tid; c < dimP; c += G_THREADS) rf[c] = expf(rf[c]);
+        for (int c = tid; c < dimP; c += G_THREADS) rf[c] = exp2f(rf[c]);
     // ---- scores: warp w takes tokens [16 (w & 3), +16) and keys [32 (w >> 2), +32)
     float s[4][4] = {};
     {
@@ -672,7 +778,7 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
                     for (int c = lane; c < dim; c += 32) {
                         const float qv = to_f32(prow[(size_t)t * a.ld + a.q_off + h * dim + c]);
                         const float kv = to_f32(prow[(size_t)key * a.ld + a.k_off + h * dim + c]);
-                        acc = fmaf(qv * kv, expf(sc.b[((size_t)(t0 + t) * a.H + h) * dim + c] - sc.b[((size_t)(t0 + key) * a.H + h) * dim + c]), acc);
+                        acc = fmaf(qv * kv, exp2f(sc.b[((size_t)(t0 + t) * a.H + h) * dim + c] - sc.b[((size_t)(t0 + key) * a.H + h) * dim + c]), acc);
                     }
                 acc = warp_sum(acc) * a.q_scale;
                 if (lane == 0) {
@@ -700,6 +806,7 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
             if (t0 + nt == cu_q[b + 1] && slot >= 0 && slot < a.n_slots) st.m[(size_t)slot * a.H + h] = Fs[nt - 1] + Ms[nt - 1];
         }
     }
+    cp_async_wait<0>();                                        // the values
     __syncthreads();
     // ---- outputs: a warp takes 16 columns of every group of 128 and every `parts`-th group of 16 tokens
     const int ncg = min(8, vdP / 16);
@@ -722,7 +829,7 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
         for (int ng = 0; ng < NG; ng++) {
             const int n0 = ng * 128 + cg * 16;
             if (n0 >= vdP) continue;
-            float x[2][4], xn[2][4];                           // S's values of a step of 16 rows: rows 2 t4, +1, +8, +9
+            float x[2][4], xn[2][4], xm[2][4];                 // S's values of a step of 16 rows: rows 2 t4, +1, +8, +9; two steps ahead
             auto fetch = [&](int k0, float (&v)[2][4]) {
 #pragma unroll
                 for (int j = 0; j < 2; j++)
@@ -733,8 +840,9 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
                     }
             };
             fetch(0, x);
+            fetch(16, xn);                                     // (rows beyond dim give zeros, without a load)
             for (int k0 = 0; k0 < dimP; k0 += 16) {
-                if (k0 + 16 < dimP) fetch(k0 + 16, xn);
+                fetch(k0 + 32, xm);
                 uint32_t bh[2][2], bl[2][2];
 #pragma unroll
                 for (int j = 0; j < 2; j++)
@@ -769,7 +877,10 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
 #pragma unroll
                 for (int j = 0; j < 2; j++)
 #pragma unroll
-                    for (int e = 0; e < 4; e++) x[j][e] = xn[j][e];
+                    for (int e = 0; e < 4; e++) {
+                        x[j][e] = xn[j][e];
+                        xn[j][e] = xm[j][e];
+                    }
             }
             if (KIND == MLSTM) {
 #pragma unroll

@@ -243,7 +243,10 @@ __device__ __forceinline__ void load8_f32(const bf16* p, float (&v)[8]) {
 }
 
 // The learned router: one CTA a token; a warp an expert's logit at a time, then one thread picks.
-constexpr int ROUTER_THREADS = 128;
+// (a step of few tokens takes CTAs of 512 threads, so that more experts' rows are in flight; a logit is one warp's sum either
+// way, so its bits do not change)
+constexpr int ROUTER_THREADS = 512;
+static int router_threads(int T, int rows) { return T <= 64 && rows > 4 ? ROUTER_THREADS : 128; }
 template <typename TA>
 __global__ void __launch_bounds__(ROUTER_THREADS)
 moe_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecRef bias, const int* __restrict__ tok_seq,
@@ -262,7 +265,7 @@ moe_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecRef bia
     const TA* x = h + (size_t)t * D;
     // rows of a multiple of 8 values go 8 values a lane and load (16 or 32 bytes), four experts of a warp in flight
     const int D8 = D % 8 == 0 ? D : 0;
-    for (int e = warp; e < E; e += ROUTER_THREADS / 32) {
+    for (int e = warp; e < E; e += (int)blockDim.x / 32) {
         const TA* wr = w + (size_t)e * D;
         float acc = 0.f;
 #pragma unroll 2
@@ -327,7 +330,7 @@ moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecR
     const TA* x = h + (size_t)t * D;
     const int D8 = D % 8 == 0 ? D : 0;
     const int n_rows = shared_gate != nullptr ? E + 1 : E;           // the shared expert's gate is one more row
-    for (int e = warp; e < n_rows; e += ROUTER_THREADS / 32) {
+    for (int e = warp; e < n_rows; e += (int)blockDim.x / 32) {
         const TA* wr = w + (size_t)e * D;
         float acc = 0.f;
 #pragma unroll 2
@@ -725,10 +728,10 @@ MYNAH_API int mynah_moe_router_ffn(const void* h, int dtype, const int* tok_seq,
     MYNAH_REQUIRE(E <= MOE_MAX_EXPERTS, "moe_router_ffn: %d experts exceed %d", E, MOE_MAX_EXPERTS);
     const VecRef bias{b_router, b_dtype};
     if (dtype == MYNAH_F32)
-        mynah_launch(moe_router_kernel<float>, dim3(T), dim3(ROUTER_THREADS), 0, stream, (const float*)h, (const float*)w_router, bias,
+        mynah_launch(moe_router_kernel<float>, dim3(T), dim3(router_threads(T, E)), 0, stream, (const float*)h, (const float*)w_router, bias,
                      tok_seq, choice, pair_weight, D, E, top);
     else if (dtype == MYNAH_BF16)
-        mynah_launch(moe_router_kernel<bf16>, dim3(T), dim3(ROUTER_THREADS), 0, stream, (const bf16*)h, (const bf16*)w_router, bias,
+        mynah_launch(moe_router_kernel<bf16>, dim3(T), dim3(router_threads(T, E)), 0, stream, (const bf16*)h, (const bf16*)w_router, bias,
                      tok_seq, choice, pair_weight, D, E, top);
     else
         return mynah_fail("moe_router_ffn: unsupported dtype %d", dtype);
@@ -759,10 +762,10 @@ MYNAH_API int mynah_moe_group_router_ffn(const void* h, int dtype, const int* to
     MYNAH_REQUIRE(shared == nullptr || shared_gate != nullptr, "moe_group_router_ffn: a shared expert's rows need its gates");
     const VecRef corr{correction, c_dtype};
     if (dtype == MYNAH_F32)
-        mynah_launch(moe_group_router_kernel<float>, dim3(T), dim3(ROUTER_THREADS), 0, stream, (const float*)h, (const float*)w_router,
+        mynah_launch(moe_group_router_kernel<float>, dim3(T), dim3(router_threads(T, E)), 0, stream, (const float*)h, (const float*)w_router,
                      corr, tok_seq, choice, pair_weight, shared_gate, D, E, top, groups, keep, weight_scale, softmax_scores, group_max);
     else if (dtype == MYNAH_BF16)
-        mynah_launch(moe_group_router_kernel<bf16>, dim3(T), dim3(ROUTER_THREADS), 0, stream, (const bf16*)h, (const bf16*)w_router,
+        mynah_launch(moe_group_router_kernel<bf16>, dim3(T), dim3(router_threads(T, E)), 0, stream, (const bf16*)h, (const bf16*)w_router,
                      corr, tok_seq, choice, pair_weight, shared_gate, D, E, top, groups, keep, weight_scale, softmax_scores, group_max);
     else
         return mynah_fail("moe_group_router_ffn: unsupported dtype %d", dtype);
