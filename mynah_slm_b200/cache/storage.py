@@ -5,7 +5,7 @@ kv_heads, 64, head_dim] in the run's type, in one allocation, and the values
 likewise with their own width and, where several key heads share a value
 head, their own number of heads (a group whose mixers keep one vector per
 position has none). Beside them: the fixed-size per-sequence state of the
-entries that ask for one, [max_seqs + 1, *shape]: a sequence's row is zeroed
+entries (and of the embedding) that ask for one, [max_seqs + 1, *shape]: a sequence's row is zeroed
 whenever its slot is handed out; the last row belongs to no sequence and is
 there for a step's padding rows.
 
@@ -53,6 +53,7 @@ class Cache:
                 self.states[i] = make(e.state)
             if getattr(e, "block_state", None) is not None:
                 self.block_states[i] = make(e.block_state)
+        self.embedding_state = make(getattr(plan, "embedding_state", None))
         self.views: list[CacheView] = []
         for i, e in enumerate(plan.entries):
             src = plan.entries[e.source] if e.source is not None else e

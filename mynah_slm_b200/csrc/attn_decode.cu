@@ -39,6 +39,7 @@ struct DecodeArgs {
     int null_key;        // 1: the softmax has one more term, of score 0 and without a value
     float out_scale;     // factor on the output rows
     int vdo;             // columns of a head in the output rows (<= VD)
+    const float* sink;   // null, or that term's score a query head (neither scaled nor capped)
 };
 
 // The pages that the query of a sequence of `hi` positions can see: pages [pg0, pg1) of the window (or of everything),
@@ -217,7 +218,7 @@ template <typename T>
 __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                            T* __restrict__ out, const int* __restrict__ kv_len, int window, int chunk,
                                            int keep_first, int H, int HD, int S_max, int ldo, int null_key, float out_scale,
-                                           int vdo) {
+                                           int vdo, const float* __restrict__ sink) {
     const int h = blockIdx.x, b = blockIdx.y;
     const size_t row0 = ((size_t)b * H + h) * S_max;
     // only the pages the sequence can see have partial results
@@ -230,7 +231,9 @@ __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o, con
         const float m = part_ml[(row0 + s) * 2];
         ls += mn == -INFINITY ? 0.f : part_ml[(row0 + s) * 2 + 1] * expf(m - mn);
     }
-    if (null_key && ls > 0.f) ls += expf(-mn);         // the term without a key; where it overflows the keys' share is zero
+    // the term without a key (score 0, or the head's sink); where it overflows the keys' share is zero
+    if (sink != nullptr && ls > 0.f) ls += expf(sink[h] - mn);
+    else if (null_key && ls > 0.f) ls += expf(-mn);
     const float inv = ls > 0.f ? out_scale / ls : 0.f;
     for (int d = threadIdx.x; d < vdo; d += blockDim.x) {
         float os = 0.f;
@@ -262,7 +265,7 @@ int launch_decode(const void* q, void* out, int B, const DecodeArgs& a, const vo
     if (mynah_check_launch("attn_decode_split")) return -1;
     const int threads = a.VD >= 128 ? 128 : (a.VD >= 64 ? 64 : 32);
     attn_decode_combine_kernel<T><<<dim3(a.H, B), threads, 0, stream>>>(part_o, part_ml, (T*)out, kv_len, a.window, a.chunk, a.keep_first, a.H, a.VD, a.S, a.ldo,
-                                                                        a.null_key, a.out_scale, a.vdo);
+                                                                        a.null_key, a.out_scale, a.vdo, a.sink);
     return mynah_check_launch("attn_decode_combine");
 }
 
@@ -296,12 +299,13 @@ MYNAH_API int mynah_attn_decode(
 
 // The same with capped scores (softcap c > 0: score <- c tanh(score / c)), first tokens that a window keeps
 // (keep_first), several key heads on one value head (the value cache has KV / vdiv heads), one more softmax term of score
-// 0 that has no value (null_key), a factor on the output (out_scale) and output heads of `vdo` columns (0: VD).
+// 0 that has no value (null_key) or of a score of its own for every query head (sink, fp32 [H]; neither scaled nor capped), a
+// factor on the output (out_scale) and output heads of `vdo` columns (0: VD).
 MYNAH_API int mynah_attn_decode_capped(
     const void* q, void* out, int dtype, int B, int H, int KV, int HD, int VD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, float out_scale, int vdo,
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, const float* sink, float out_scale, int vdo,
     int n_splits, float* scratch, int* status, cudaStream_t stream);
 
 MYNAH_API int mynah_attn_decode_ex(
@@ -310,14 +314,14 @@ MYNAH_API int mynah_attn_decode_ex(
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
     int window, int chunk, float scale, int n_splits, float* scratch, int* status, cudaStream_t stream) {
     return mynah_attn_decode_capped(q, out, dtype, B, H, KV, HD, VD, ldq, ldo, k_cache, v_cache, kv_len, page_indptr, page_ids,
-                                    page_base, n_pages, window, chunk, scale, 0.f, 0, 1, 0, 1.0f, VD, n_splits, scratch, status, stream);
+                                    page_base, n_pages, window, chunk, scale, 0.f, 0, 1, 0, nullptr, 1.0f, VD, n_splits, scratch, status, stream);
 }
 
 MYNAH_API int mynah_attn_decode_capped(
     const void* q, void* out, int dtype, int B, int H, int KV, int HD, int VD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, float out_scale, int vdo,
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, const float* sink, float out_scale, int vdo,
     int n_splits, float* scratch, int* status, cudaStream_t stream) {
     if (B == 0) return 0;
     MYNAH_REQUIRE(softcap >= 0.f && keep_first >= 0 && vdiv >= 1 && KV % vdiv == 0, "attn_decode: bad cap, kept tokens or value sharing");
@@ -334,7 +338,7 @@ MYNAH_API int mynah_attn_decode_capped(
     int lpk = 1;
     while (lpk * 8 < HD || lpk * 8 < VD) lpk <<= 1;
     const DecodeArgs a{H, KV, HD, ldq, ldo, window, n_splits, lpk, scale != 0.f ? scale : 1.0f / sqrtf((float)HD), VD, chunk, softcap, keep_first, vdiv,
-                       null_key, out_scale, vdo > 0 ? vdo : VD};
+                       null_key, out_scale, vdo > 0 ? vdo : VD, sink};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     float* part_o = scratch;
     float* part_ml = scratch + (size_t)B * H * n_splits * VD;

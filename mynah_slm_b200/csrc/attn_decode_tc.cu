@@ -70,6 +70,7 @@ struct TcArgs {
     int null_key = 0;       // 1: the softmax has one more term, of score 0 and without a value (the merge adds it)
     float out_scale = 1.f;  // factor on the output rows
     int vdo = 0;            // columns of a head in the output rows; 0: the value head's width
+    const float* sink = nullptr;   // null, or the further term's score a query head (the merge adds it)
 };
 
 // The pages that a sequence's newest position sees: pages [pg0, pg1) of its window (or of everything), and before them
@@ -371,7 +372,8 @@ __device__ __forceinline__ void compute_page(const PageJob& job, const uint32_t 
 // pays the chain of dependent reads that finds its next page.)
 template <int HD> __device__ __forceinline__ void merge_pages(const float* __restrict__, const float* __restrict__, bf16* __restrict__,
                                                               size_t, int, int, int, float*, float*, float*,
-                                                                       int null_key = 0, float out_scale = 1.f, int vdo = HD);
+                                                                       int null_key = 0, float out_scale = 1.f, int vdo = HD,
+                                                                       const float* __restrict__ sink = nullptr);
 
 // MERGE: the CTA that finishes a (sequence, kv head) last also merges its pages (a count per pair, zero before the
 // first launch and left zero by every launch), which saves the merge's launch; without it the merge is a launch
@@ -426,7 +428,8 @@ attn_decode_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
 template <int HD>
 __device__ __forceinline__ void merge_pages(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                             bf16* __restrict__ out_row, size_t r0g, int G, int S, int n_vis,
-                                            float* w_s, float* acc_s, float* inv_s, int null_key, float out_scale, int vdo) {
+                                            float* w_s, float* acc_s, float* inv_s, int null_key, float out_scale, int vdo,
+                                            const float* __restrict__ sink) {
     // (G may also be 1 with r0g and out_row pointing at one head: a head's arithmetic does not involve the others.)
     constexpr int LPR = HD / 4, NS = WARPS * 32 / LPR;
     constexpr int AHEAD = 8;                          // output rows a thread fetches before it has their weights
@@ -469,8 +472,10 @@ __device__ __forceinline__ void merge_pages(const float* __restrict__ part_o, co
             ls = fmaf(ml.y, w, ls);
         }
         ls = warp_sum(ls);
-        // the term without a key counts exp(0 - max); where that overflows, the keys' share of the softmax is zero
-        if (null_key && ls > 0.f) ls += expf(-mmax);
+        // the term without a key counts exp(0 - max), or exp(sink - max) with a sink for every head of the call; where that
+        // overflows, the keys' share of the softmax is zero
+        if (sink != nullptr && ls > 0.f) ls += expf(sink[i] - mmax);
+        else if (null_key && ls > 0.f) ls += expf(-mmax);
         if (lane == 0) inv_s[i] = ls > 0.f ? out_scale / ls : 0.f;
     }
     __syncthreads();
@@ -509,7 +514,7 @@ template <int HD>
 __global__ void __launch_bounds__(WARPS * 32)
 attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out,
                          const int* __restrict__ kv_len, int window, int keep_first, int H, int S, int ldo,
-                         int null_key, float out_scale, int vdo) {
+                         int null_key, float out_scale, int vdo, const float* __restrict__ sink) {
     constexpr int NS = WARPS * 32 / (HD / 4);
     extern __shared__ float w_s[];
     __shared__ __align__(16) float acc_s[NS * HD];
@@ -520,7 +525,7 @@ attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restri
     const int hi = kv_len[b];
     const int n_vis = min(S, visible_pages(hi, window, keep_first).count());
     merge_pages<HD>(part_o, part_ml, out + (size_t)b * ldo + (size_t)h * vdo, ((size_t)b * H + h) * S, 1, S, n_vis, w_s, acc_s, inv_s,
-                    null_key, out_scale, vdo);
+                    null_key, out_scale, vdo, sink != nullptr ? sink + h : nullptr);
 }
 
 // ---------------------------------------------------------------------------------------------------------
@@ -962,7 +967,7 @@ MYNAH_API int mynah_attn_decode_tc_capped(
     const void* q, void* out, int B, int H, int KV, int HD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window_in, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, float out_scale, int vdo,
+    int window_in, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, const float* sink, float out_scale, int vdo,
     int n_splits, float* scratch, unsigned* counters, int* status, cudaStream_t stream);
 
 // The same with a chunk mask instead of the window (one of the two, 0: none) and a score scale given by the caller
@@ -973,26 +978,26 @@ MYNAH_API int mynah_attn_decode_tc_ex(
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
     int window_in, int chunk, float scale, int n_splits, float* scratch, unsigned* counters, int* status, cudaStream_t stream) {
     return mynah_attn_decode_tc_capped(q, out, B, H, KV, HD, ldq, ldo, k_cache, v_cache, kv_len, page_indptr, page_ids, page_base,
-                                       n_pages, window_in, chunk, scale, 0.f, 0, 1, HD, 0, 1.0f, HD, n_splits, scratch, counters, status, stream);
+                                       n_pages, window_in, chunk, scale, 0.f, 0, 1, HD, 0, nullptr, 1.0f, HD, n_splits, scratch, counters, status, stream);
 }
 
 // The same with capped scores (softcap c > 0: score <- c tanh(score / c), after the scale), first tokens that the window
 // keeps (keep_first, with a window and no chunk; the page lists must then hold every page of a sequence) and `vdiv` key
 // heads on one value head (the value cache is [n_pages, KV / vdiv, 64, VD]), value heads of a width VD of their own (64 or
-// 128; scratch of B * H * n_splits * (VD + 2) floats), one more softmax term of score 0 that has no value (null_key), a factor
-// on the output (out_scale) and output heads of `vdo` columns (at most VD: padding columns of the values are left out).
+// 128; scratch of B * H * n_splits * (VD + 2) floats), one more softmax term of score 0 that has no value (null_key)
+// or of a score of its own for every query head (sink, fp32 [H]; neither scaled nor capped), a factor on the output (out_scale) and output heads of `vdo` columns (at most VD: padding columns of the values are left out).
 MYNAH_API int mynah_attn_decode_tc_capped(
     const void* q, void* out, int B, int H, int KV, int HD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window_in, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, float out_scale, int vdo,
+    int window_in, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, const float* sink, float out_scale, int vdo,
     int n_splits, float* scratch, unsigned* counters, int* status, cudaStream_t stream) {
     if (B == 0) return 0;
     MYNAH_REQUIRE(window_in >= 0 && chunk >= 0 && !(window_in > 0 && chunk > 0), "attn_decode_tc: a window or a chunk, not both");
     MYNAH_REQUIRE(softcap >= 0.f && keep_first >= 0 && vdiv >= 1 && KV % vdiv == 0 && (keep_first == 0 || chunk == 0),
                   "attn_decode_tc: bad cap, kept tokens or value sharing");
     MYNAH_REQUIRE((VD == 64 || VD == 128) && vdo > 0 && vdo <= VD, "attn_decode_tc: value heads of %d with %d output columns are not taken by this kernel", VD, vdo);
-    MYNAH_REQUIRE(counters == nullptr || (VD == HD && vdo == VD && !null_key && out_scale == 1.0f),
+    MYNAH_REQUIRE(counters == nullptr || (VD == HD && vdo == VD && !null_key && sink == nullptr && out_scale == 1.0f),
                   "attn_decode_tc: the merging form takes plain heads of one width");
     const int window = chunk > 0 ? -chunk : window_in;
     MYNAH_REQUIRE(mynah_attn_decode_tc_supported(H, KV, HD), "attn_decode_tc: H=%d KV=%d head_dim=%d is not taken by this kernel", H, KV, HD);
@@ -1000,7 +1005,7 @@ MYNAH_API int mynah_attn_decode_tc_capped(
     MYNAH_REQUIRE(n_splits >= 1 && n_splits <= 65535 && B <= 65535 && KV <= 65535, "attn_decode_tc: launch too large");
     MYNAH_REQUIRE(scratch != nullptr, "attn_decode_tc: no scratch memory given");
     const TcArgs a{H, KV, ldq, window, n_splits, scale != 0.f ? scale : 1.0f / sqrtf((float)HD), window > 0 ? keep_first : 0, vdiv, softcap,
-                   null_key, out_scale, vdo};
+                   null_key, out_scale, vdo, sink};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     float* part_o = scratch;
     float* part_ml = scratch + (size_t)B * H * n_splits * VD;
@@ -1047,10 +1052,10 @@ MYNAH_API int mynah_attn_decode_tc_capped(
     MYNAH_REQUIRE(dyn <= MERGE_MAX_BYTES, "attn_decode_tc: %d pages a sequence exceed what the merge holds", n_splits);
     if (VD == 128)
         mynah_launch(attn_decode_merge_kernel<128>, dim3(H, B), dim3(WARPS * 32), dyn, stream, part_o, part_ml, (bf16*)out, kv_len, window, a.keep_first, H, n_splits, ldo,
-                     null_key, out_scale, vdo);
+                     null_key, out_scale, vdo, sink);
     else
         mynah_launch(attn_decode_merge_kernel<64>, dim3(H, B), dim3(WARPS * 32), dyn, stream, part_o, part_ml, (bf16*)out, kv_len, window, a.keep_first, H, n_splits, ldo,
-                     null_key, out_scale, vdo);
+                     null_key, out_scale, vdo, sink);
     return mynah_check_launch("attn_decode_merge");
 }
 
@@ -1092,9 +1097,9 @@ MYNAH_API int mynah_attn_decode_fused(
         if (mynah_check_launch("attn_decode_fused (pages)")) return -1;
         const size_t dyn_m = (size_t)n_splits * sizeof(float);
         if (HD == 128)
-            mynah_launch(attn_decode_merge_kernel<128>, dim3(H, B), dim3(WARPS * 32), dyn_m, stream, part_o, part_ml, (bf16*)out, kv_len, window, 0, H, n_splits, ldo, 0, 1.0f, HD);
+            mynah_launch(attn_decode_merge_kernel<128>, dim3(H, B), dim3(WARPS * 32), dyn_m, stream, part_o, part_ml, (bf16*)out, kv_len, window, 0, H, n_splits, ldo, 0, 1.0f, HD, (const float*)nullptr);
         else
-            mynah_launch(attn_decode_merge_kernel<64>, dim3(H, B), dim3(WARPS * 32), dyn_m, stream, part_o, part_ml, (bf16*)out, kv_len, window, 0, H, n_splits, ldo, 0, 1.0f, HD);
+            mynah_launch(attn_decode_merge_kernel<64>, dim3(H, B), dim3(WARPS * 32), dyn_m, stream, part_o, part_ml, (bf16*)out, kv_len, window, 0, H, n_splits, ldo, 0, 1.0f, HD, (const float*)nullptr);
         return mynah_check_launch("attn_decode_merge");
     }
     if (HD == 128)

@@ -36,6 +36,7 @@ struct PrefillArgs {
     int null_key;               // 1: the softmax has one more term, of score 0 and without a value
     float out_scale;            // factor on the output rows
     int vdo;                    // columns of a head in the output rows (<= VD: padding columns of the values are left out)
+    const float* sink;          // null, or that term's score a query head (neither scaled nor capped)
 };
 
 template <typename TA, typename TC>
@@ -145,8 +146,10 @@ attn_prefill_generic_kernel(const TA* __restrict__ q, TA* __restrict__ out,
     for (int i = 0; i < QPW; i++) {
         const int qi = warp * QPW + i;
         if (qi >= nq) continue;
-        // the term without a key counts exp(0 - m); where that overflows, the keys' share of the softmax is zero
-        const float ls = a.null_key && l[i] > 0.f ? l[i] + expf(-m[i]) : l[i];
+        // the term without a key counts exp(0 - m), or exp(sink - m); where that overflows, the keys' share of the softmax is zero
+        float ls = l[i];
+        if (a.sink != nullptr && ls > 0.f) ls += expf(a.sink[h] - m[i]);
+        else if (a.null_key && ls > 0.f) ls += expf(-m[i]);
         const float inv = ls > 0.f ? a.out_scale / ls : 0.f;
         TA* o = out + (size_t)(q0 + tile0 + qi) * a.ldo + (size_t)h * a.vdo;
 #pragma unroll
@@ -169,12 +172,13 @@ MYNAH_API int mynah_attn_prefill_generic_ex(
 
 // The same with capped scores (softcap c > 0: score <- c tanh(score / c)), first tokens that a window keeps
 // (keep_first), several key heads on one value head (the value cache has KV / vdiv heads), one more softmax term of score
-// 0 that has no value (null_key), a factor on the output (out_scale) and output heads of `vdo` columns (0: VD).
+// 0 that has no value (null_key) or of a score of its own for every query head (sink, fp32 [H]; neither scaled nor capped), a
+// factor on the output (out_scale) and output heads of `vdo` columns (0: VD).
 MYNAH_API int mynah_attn_prefill_generic_capped(
     const void* q, void* out, int dtype, int n_tokens, int B, int max_q_len, int H, int KV, int HD, int VD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* cu_q, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, float out_scale, int vdo,
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, const float* sink, float out_scale, int vdo,
     int* status, cudaStream_t stream);
 
 // q: [T, ldq] with head h at columns [h*HD, (h+1)*HD); out: [T, ldo] likewise.
@@ -195,14 +199,14 @@ MYNAH_API int mynah_attn_prefill_generic_ex(
     int window, int chunk, float scale, int* status, cudaStream_t stream) {
     return mynah_attn_prefill_generic_capped(q, out, dtype, n_tokens, B, max_q_len, H, KV, HD, VD, ldq, ldo, k_cache, v_cache,
                                              cu_q, kv_len, page_indptr, page_ids, page_base, n_pages, window, chunk, scale,
-                                             0.f, 0, 1, 0, 1.0f, VD, status, stream);
+                                             0.f, 0, 1, 0, nullptr, 1.0f, VD, status, stream);
 }
 
 MYNAH_API int mynah_attn_prefill_generic_capped(
     const void* q, void* out, int dtype, int n_tokens, int B, int max_q_len, int H, int KV, int HD, int VD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* cu_q, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, float out_scale, int vdo,
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int null_key, const float* sink, float out_scale, int vdo,
     int* status, cudaStream_t stream) {
     if (B == 0 || max_q_len == 0) return 0;
     MYNAH_REQUIRE(softcap >= 0.f && keep_first >= 0 && vdiv >= 1 && KV % vdiv == 0, "attn_prefill: bad cap, kept tokens or value sharing");
@@ -215,7 +219,7 @@ MYNAH_API int mynah_attn_prefill_generic_capped(
     MYNAH_REQUIRE(H <= 65535, "attn_prefill: H=%d exceeds one launch", H);
     MYNAH_REQUIRE(window >= 0, "attn_prefill: negative window");
     const PrefillArgs a{B, H, KV, HD, ldq, ldo, window, scale != 0.f ? scale : 1.0f / sqrtf((float)HD), VD, chunk, softcap, keep_first, vdiv,
-                        null_key, out_scale, vdo > 0 ? vdo : VD};
+                        null_key, out_scale, vdo > 0 ? vdo : VD, sink};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     const size_t smem = sizeof(float) * ((size_t)KT * (HD + 1) + (size_t)KT * VD + (size_t)QT * HD);
     (void)max_q_len;

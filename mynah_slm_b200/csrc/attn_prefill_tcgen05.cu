@@ -54,6 +54,7 @@ struct PfArgs {
     int null_key;                     // 1: the softmax has one more term, of score 0 and without a value
     float out_scale;                  // factor on the output rows
     int vdo;                          // columns of a head in the output rows (a multiple of 8, at most VD)
+    const float* sink;                // null, or that term's score a query head (neither scaled nor capped)
     float cap_in, cap_log2;           // capped scores (CAP kernels): c tanh(s scale / c) log2(e) = cap_log2 * tanh(s * cap_in)
     // The first key that the row at position p sees. Window and chunk both give a bound that does not fall as p
     // grows, so a tile's first row has the tile's lowest bound and its last row the highest.
@@ -501,8 +502,9 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (ok && !warp_wait(o_done, (n_tiles - 1) & 1)) ok = false;
         if (ok) {
             tc_fence_after();
-            // the term without a key counts 2^(0 - m); where that overflows, the keys' share of the softmax is zero
-            if (a.null_key && l > 0.f) l += ex2(-m_ref);
+            // the term without a key counts 2^(0 - m), or 2^(sink log2(e) - m); where that overflows, the keys' share of the softmax is zero
+            if (a.sink != nullptr && l > 0.f) l += ex2(fmaf(a.sink[h], 1.4426950408889634f, -m_ref));
+            else if (a.null_key && l > 0.f) l += ex2(-m_ref);
             const float inv = l > 0.f ? a.out_scale / l : 0.f;
             bf16* o_row = out + (size_t)(q_begin + q0 + row) * a.ldo + (size_t)h * a.vdo + grp * (VD / 2);
 #pragma unroll 1
@@ -606,7 +608,7 @@ MYNAH_API int mynah_attn_prefill_tcgen05_capped(
     const void* q, void* out, int n_tokens, int B, int max_q_len, int H, int KV, int HD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* cu_q, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, float out_scale, int vdo,
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, const float* sink, float out_scale, int vdo,
     int* status, cudaStream_t stream);
 
 // The same with a chunk mask beside the window (0: none) and a score scale given by the caller (0: 1/sqrt(HD)).
@@ -616,19 +618,20 @@ MYNAH_API int mynah_attn_prefill_tcgen05_ex(
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
     int window, int chunk, float scale, int* status, cudaStream_t stream) {
     return mynah_attn_prefill_tcgen05_capped(q, out, n_tokens, B, max_q_len, H, KV, HD, ldq, ldo, k_cache, v_cache, cu_q, kv_len,
-                                             page_indptr, page_ids, page_base, n_pages, window, chunk, scale, 0.f, 0, 1, HD, 0, 1.0f, HD, status, stream);
+                                             page_indptr, page_ids, page_base, n_pages, window, chunk, scale, 0.f, 0, 1, HD, 0, nullptr, 1.0f, HD, status, stream);
 }
 
 // The same with capped scores (softcap c > 0: score <- c tanh(score / c), after the scale), first tokens that the window
 // keeps (keep_first; the page lists must then hold every page of a sequence) and `vdiv` key heads on one value head (the
 // value cache is [n_pages, KV / vdiv, 64, VD]), value heads of a width VD of their own (64 or 128), one more softmax term of
-// score 0 that has no value (null_key), a factor on the output (out_scale) and output heads of `vdo` columns (a multiple of 8
+// score 0 that has no value (null_key) or of a score of its own for every query head (sink, fp32 [H]; neither scaled nor capped),
+// a factor on the output (out_scale) and output heads of `vdo` columns (a multiple of 8
 // up to VD: the padding columns of the values are left out).
 MYNAH_API int mynah_attn_prefill_tcgen05_capped(
     const void* q, void* out, int n_tokens, int B, int max_q_len, int H, int KV, int HD, int ldq, int ldo,
     const void* k_cache, const void* v_cache, const int* cu_q, const int* kv_len,
     const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, float out_scale, int vdo,
+    int window, int chunk, float scale, float softcap, int keep_first, int vdiv, int VD, int null_key, const float* sink, float out_scale, int vdo,
     int* status, cudaStream_t stream) {
     if (B == 0 || max_q_len == 0 || n_tokens == 0) return 0;
     MYNAH_REQUIRE(window >= 0 && chunk >= 0, "attn_prefill_tcgen05: negative window or chunk");
@@ -648,7 +651,7 @@ MYNAH_API int mynah_attn_prefill_tcgen05_capped(
     if (make_map(&mv, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (long long)n_pages * (KV / vdiv) * PAGE_TOKENS, VD, VD, PAGE_TOKENS, 64)) return -1;
     const float scale_used = scale != 0.f ? scale : 1.0f / sqrtf((float)HD);
     const PfArgs a{B, H, KV, ldo, window, scale_used * 1.4426950408889634f, chunk, keep_first, vdiv,
-                   null_key, out_scale, vdo, softcap > 0.f ? scale_used / softcap : 0.f, softcap * 1.4426950408889634f};
+                   null_key, out_scale, vdo, sink, softcap > 0.f ? scale_used / softcap : 0.f, softcap * 1.4426950408889634f};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     // Two CTAs an SM pay once there are several waves of CTAs (64 prompts of 2,048 tokens and 32 heads: 2.97 against
     // 3.34 ms; 4 prompts: 221 against 236 us); with one wave or two, the longest CTA's own chain sets the time and it

@@ -3,7 +3,7 @@
 //   q <- q / rms(q over all heads) * wq          (one RMS over the H*dim outputs, gain of that size; k likewise)
 //   rotary positions on the first `rot` dimensions of each head of q and k, element i paired with i + rot/2:
 //       (u, v) -> (u cos a - v sin a, v cos a + u sin a),   a = position * base^(-2i/rot)   (tables built in double)
-//   v <- v / rms(v over the head's vd values)     (no gain)
+//   v <- v / rms(v over the head's vd values)     (no gain; optional)
 //   v <- (1 - lambda) v + lambda v_first          (optional: v_first holds the same token's values of an earlier
 //                                                  layer, written here by the layer that comes first)
 //   q -> q_out, k and v -> the paged cache
@@ -19,6 +19,7 @@ struct PrepArgs {
     int H, G, dim, vd, dimp, vdp, ld, ldq, rot, n_pos;
     float eps;
     int vmix;        // 0: none, 1: write v_first, 2: mix with v_first
+    int vnorm;       // 1: values are normed
     int vec;         // 1: the q and k heads go eight elements a thread (see norm_rotate_heads8)
 };
 
@@ -164,7 +165,7 @@ attn_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw, Ve
             const float v = to_f32(vsrc[g * a.vd + d]);
             sv = fmaf(v, v, sv);
         }
-        const float rv = 1.0f / sqrtf(warp_sum(sv) / (float)a.vd + a.eps);
+        const float rv = a.vnorm ? 1.0f / sqrtf(warp_sum(sv) / (float)a.vd + a.eps) : 1.0f;
         T* dst = v_cache + (((size_t)page * a.G + g) * PAGE_TOKENS + in_page) * a.vdp;
         float* vf = v_first ? v_first + ((size_t)row * a.G + g) * a.vd : nullptr;
         for (int d = lane; d < a.vdp; d += 32) {
@@ -179,10 +180,10 @@ attn_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw, Ve
     }
 }
 
-// The vector form of the whole kernel (taken when `vec` holds and the values fit too: vd % 8 == 0, vdp == vd, at most
-// 8 * 1024 elements a row): a thread fetches its eight-element pieces of q, k and v at once, the three kinds of
-// sums of squares are formed together (q and k over the block, a value head over the lanes that hold it: vd / 8, a
-// power of two up to 32), and every piece is normed, rotated with its partner piece (fetched again from L1) and stored.
+// The vector form of the whole kernel (taken when heads of q, k and v are whole 16-byte pieces, rot % 16 == 0 and a row has at
+// most 8 * 1024 elements; stored heads may be wider, the columns behind the head are zeros): a thread fetches its eight-element pieces of q, k and v at once, the three kinds of
+// sums of squares are formed together (q and k over the block, a value head that is normed over the lanes that hold it:
+// vd / 8, a power of two up to 32), and every piece is normed, rotated with its partner piece (fetched again from L1) and stored.
 template <typename T>
 __global__ void __launch_bounds__(1024)
 attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw, VecRef kw,
@@ -202,7 +203,7 @@ attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw
     const int n_all = nq + (writes ? nk + nv : 0);
     if (b < 0) {
         float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        if (i < nq) store8(qo + i, zero);
+        for (int j = i; j < a.H * a.dimp; j += blockDim.x * 8) store8(qo + j, zero);
         return;
     }
     const int pos = tok_pos[row];
@@ -227,7 +228,7 @@ attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     // a value head lies in vd / 8 consecutive threads of one warp (its start is a multiple of vd / 8 pieces)
     float sv = ss;
-    for (int o = (a.vd >> 3) >> 1; o > 0; o >>= 1) sv += __shfl_xor_sync(0xffffffffu, sv, o);
+    if (a.vnorm) for (int o = (a.vd >> 3) >> 1; o > 0; o >>= 1) sv += __shfl_xor_sync(0xffffffffu, sv, o);
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     if (lane == 0) {
@@ -274,7 +275,7 @@ attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw
     } else if (is_v) {
         const int local = i - nq - nk;
         const int g = local / a.vd, d = local % a.vd;
-        const float rv = 1.0f / sqrtf(sv / (float)a.vd + a.eps);
+        const float rv = a.vnorm ? 1.0f / sqrtf(sv / (float)a.vd + a.eps) : 1.0f;
         float out[8];
 #pragma unroll
         for (int e = 0; e < 8; e++) out[e] = x[e] * rv;
@@ -289,20 +290,28 @@ attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw
         }
         store8(v_cache + (((size_t)page * a.G + g) * PAGE_TOKENS + pos % PAGE_TOKENS) * a.vdp + d, out);
     }
+    // the columns behind the heads
+    const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    const int kp = (a.dimp - a.dim) >> 3, vp = (a.vdp - a.vd) >> 3;
+    for (int j = threadIdx.x; j < a.H * kp; j += blockDim.x) store8(qo + (j / kp) * a.dimp + a.dim + (j % kp) * 8, zero);
+    if (!writes) return;
+    const size_t at = (size_t)page * a.G * PAGE_TOKENS + pos % PAGE_TOKENS;
+    for (int j = threadIdx.x; j < a.G * kp; j += blockDim.x) store8(k_cache + (at + (size_t)(j / kp) * PAGE_TOKENS) * a.dimp + a.dim + (j % kp) * 8, zero);
+    for (int j = threadIdx.x; j < a.G * vp; j += blockDim.x) store8(v_cache + (at + (size_t)(j / vp) * PAGE_TOKENS) * a.vdp + a.vd + (j % vp) * 8, zero);
 }
 
 }  // namespace
 
 // qkv [T, ld]: H*dim query, then G*dim key, then G*vd value outputs a row. q_out [T, ldq] with head h at
 // h*dimp. Caches [n_pages][G][PAGE_TOKENS][dimp | vdp]; null caches: only q is made. cos/sin [n_pos, rot/2]
-// fp32 (rot 0: no rotation). v_first fp32 [T, G*vd]; lambda: one fp32 on the device.
+// fp32 (rot 0: no rotation). v_first fp32 [T, G*vd]; lambda: one fp32 on the device. vnorm 0: the values are cached as projected.
 MYNAH_API int mynah_attn_prep(const void* qkv, int dtype, int T, int ld, void* q_out, int ldq,
                               int H, int G, int dim, int vd, int dimp, int vdp,
                               const void* q_gain, const void* k_gain, int gain_dtype, float eps,
                               const float* cos_t, const float* sin_t, int rot, int n_pos,
                               const int* tok_seq, const int* tok_pos,
                               const int* page_indptr, const int* page_ids, const int* page_base, int n_pages,
-                              void* k_cache, void* v_cache, float* v_first, const float* lambda_p, int vmix,
+                              void* k_cache, void* v_cache, float* v_first, const float* lambda_p, int vmix, int vnorm,
                               int* status, cudaStream_t stream) {
     if (T == 0) return 0;
     MYNAH_REQUIRE(T > 0 && H > 0 && G > 0 && dim > 0 && vd > 0, "attn_prep: bad sizes T=%d H=%d G=%d dim=%d vd=%d", T, H, G, dim, vd);
@@ -313,14 +322,16 @@ MYNAH_API int mynah_attn_prep(const void* qkv, int dtype, int T, int ld, void* q
     MYNAH_REQUIRE((k_cache == nullptr) == (v_cache == nullptr), "attn_prep: keys and values are cached together");
     MYNAH_REQUIRE(vmix == 0 || (v_first != nullptr && (vmix == 1 || lambda_p != nullptr)), "attn_prep: value mixing needs its buffers");
     auto fits = [](const void* p) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) & 31) == 0; };
-    const int vec = dim % 8 == 0 && dimp == dim && rot % 16 == 0 && ld % 8 == 0 && ldq % 8 == 0 && fits(qkv) && fits(q_out) &&
-                    fits(q_gain) && fits(k_gain) && fits(cos_t) && fits(sin_t) && fits(k_cache);
-    const PrepArgs a{H, G, dim, vd, dimp, vdp, ld, ldq, rot, n_pos, eps, vmix, vec};
+    const bool whole = dim % 8 == 0 && dimp % 8 == 0 && rot % 16 == 0 && ld % 8 == 0 && ldq % 8 == 0 && fits(qkv) && fits(q_out) &&
+                       fits(q_gain) && fits(k_gain) && fits(cos_t) && fits(sin_t) && fits(k_cache);
+    const int vec = whole && dimp == dim;
+    const PrepArgs a{H, G, dim, vd, dimp, vdp, ld, ldq, rot, n_pos, eps, vmix, vnorm, vec};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     const VecRef qw{q_gain, gain_dtype}, kw{k_gain, gain_dtype};
     const int vd8 = vd / 8;
-    const bool one_phase = vec && vd % 8 == 0 && vdp == vd && (vd8 & (vd8 - 1)) == 0 && vd8 <= 32 && fits(v_cache) && fits(v_first) &&
-                           H * dim + G * dim + G * vd <= 8 * 1024 && ((H + G) * dim / 8) % vd8 == 0 &&
+    const bool v_lanes = !vnorm || ((vd8 & (vd8 - 1)) == 0 && vd8 <= 32 && ((H + G) * dim / 8) % vd8 == 0);
+    const bool one_phase = whole && vd % 8 == 0 && vdp % 8 == 0 && v_lanes && fits(v_cache) && fits(v_first) &&
+                           H * dim + G * dim + G * vd <= 8 * 1024 &&
                            (dtype == MYNAH_F32 || dtype == MYNAH_BF16);
     if (one_phase) {
         const int n_all = H * dim + (k_cache ? G * (dim + vd) : 0);

@@ -5,6 +5,7 @@
 // scale are fp32; the order of every sum is fixed by the thread layout, so a
 // row's result does not depend on which other rows share the launch.
 #include "common.cuh"
+#include "layout.cuh"
 #include "head_prep.cuh"
 
 // ------------------------------------------------------------- embedding
@@ -38,6 +39,66 @@ MYNAH_API int mynah_embed_gather(const void* table, int table_dtype, const int* 
     else
         return mynah_fail("embed_gather: unsupported table dtype %d", table_dtype);
     return mynah_check_launch("embed_gather");
+}
+
+// x[t, :] = E[token_t, :] + P[row_t, :] with row_t = (token before * mul_prev + token_t * mul_cur) mod buckets, and row_t =
+// buckets for a sequence's first token. The token before is the row above, or, for the first row of a sequence's piece, what
+// the sequence's last step left in last_token[slot]; that row's CTA then leaves the piece's last token there (no other CTA
+// touches the entry, so the read and the write are ordered inside one thread).
+template <typename TW>
+__global__ void embed_pairs_kernel(const TW* __restrict__ table, const TW* __restrict__ pairs, const int* __restrict__ tokens,
+                                   const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ cu_q,
+                                   const int* __restrict__ slots, int* __restrict__ last_token, float* __restrict__ x, int D, int V,
+                                   int n_slots, int buckets, long long mul_prev, long long mul_cur, int* __restrict__ status) {
+    __shared__ int row_s;
+    griddep_launch_small();
+    griddep_wait();
+    const int t = blockIdx.x, b = tok_seq[t];
+    float* out = x + (size_t)t * D;
+    const int tok = tokens[t];
+    if (b < 0 || tok < 0 || tok >= V) {      // a padding row (or an id that the host refuses already)
+        for (int i = threadIdx.x; i < D; i += blockDim.x) out[i] = 0.f;
+        return;
+    }
+    if (threadIdx.x == 0) {
+        const int slot = slots[b], q0 = cu_q[b];
+        const bool live = slot >= 0 && slot < n_slots;
+        int before = t > q0 ? tokens[t - 1] : (live ? last_token[slot] : 0);
+        if (t == q0 && live) last_token[slot] = tokens[cu_q[b + 1] - 1];
+        int row = buckets;
+        if (tok_pos[t] > 0) {
+            if (before < 0 || before >= V) {
+                atomicOr(status, MYNAH_ST_TOKEN_RANGE);
+                before = 0;
+            }
+            // both products reduced before they are added: no overflow for any ids and multipliers of 31 bits
+            row = (int)(((long long)before * mul_prev % buckets + (long long)tok * mul_cur % buckets) % buckets);
+        }
+        row_s = row;
+    }
+    __syncthreads();
+    const TW* er = table + (size_t)tok * D;
+    const TW* pr = pairs + (size_t)row_s * D;
+    for (int i = threadIdx.x; i < D; i += blockDim.x) out[i] = to_f32(er[i]) + to_f32(pr[i]);
+}
+
+// table [V][D], pairs [buckets + 1][D], both in table_dtype; last_token int32 [n_slots + 1], kept from step to step.
+MYNAH_API int mynah_embed_pairs(const void* table, const void* pairs, int table_dtype, const int* tokens, const int* tok_seq, const int* tok_pos,
+                                const int* cu_q, const int* slots, int* last_token, float* x, int T, int D, int V, int n_slots, int buckets,
+                                long long mul_prev, long long mul_cur, int* status, cudaStream_t stream) {
+    if (T == 0) return 0;
+    MYNAH_REQUIRE(T > 0 && D > 0 && V > 0 && buckets > 0, "embed_pairs: bad sizes T=%d D=%d V=%d buckets=%d", T, D, V, buckets);
+    MYNAH_REQUIRE(mul_prev >= 0 && mul_cur >= 0 && mul_prev < (1ll << 31) && mul_cur < (1ll << 31), "embed_pairs: the multipliers must lie in 0 .. 2^31 - 1");
+    const int threads = D >= 1024 ? 256 : (D >= 256 ? 128 : 64);
+    if (table_dtype == MYNAH_F32)
+        mynah_launch(embed_pairs_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)table, (const float*)pairs, tokens, tok_seq, tok_pos,
+                     cu_q, slots, last_token, x, D, V, n_slots, buckets, mul_prev, mul_cur, status);
+    else if (table_dtype == MYNAH_BF16)
+        mynah_launch(embed_pairs_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16*)table, (const bf16*)pairs, tokens, tok_seq, tok_pos,
+                     cu_q, slots, last_token, x, D, V, n_slots, buckets, mul_prev, mul_cur, status);
+    else
+        return mynah_fail("embed_pairs: unsupported table dtype %d", table_dtype);
+    return mynah_check_launch("embed_pairs");
 }
 
 // --------------------------------------------------------------- RMSNorm

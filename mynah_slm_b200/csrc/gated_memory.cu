@@ -1,4 +1,4 @@
-// Linear attention with learned decays, in two kinds. Per head, with S [dim x vd] the state (fp32, per slot) and
+// Linear attention with decays, in three kinds. Per head, with S [dim x vd] the state (fp32, per slot) and
 // k, q, v the token's rows (q times q_scale):
 //
 //   GLA     S_t = diag(a_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   a_t = sigmoid(z_t)^(1/tau) a key channel,
@@ -6,9 +6,10 @@
 //   MLSTM   (the matrix memory of xLSTM) log gates i = cap tanh((p_i + b_i)/cap), f = log sigmoid(cap tanh((p_f + b_f)/cap));
 //           m_t = max(f + m_(t-1), i)  (from m = 0);  S and n decay by exp(f + m_(t-1) - m_t) and take exp(i - m_t) k v^T
 //           (n: the same with k alone);   o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + 1e-6)
+//   FIXED   (retention) S_t = decay_head S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t
 //
-// and behind either, in the same kernel:  out = o / sqrt(mean(o^2) + eps) * w[head, column] * act(gate),  act silu (GLA) or
-// sigmoid (MLSTM), written in the rows' type to `out`'s columns [o_off + head * vd, ...).
+// and behind either, in the same kernel:  out = o / sqrt(mean(o^2) + eps) * w[head, column] * act(gate),  act silu (GLA, FIXED)
+// or sigmoid (MLSTM), written in the rows' type to `out`'s columns [o_off + head * vd, ...).
 //
 // Token form (gm_token): a CTA takes a head of a sequence and walks its tokens; a thread owns fixed entries of S. One token a
 // sequence (a decode step): S passes once through registers, from memory and back. Several: S stays in shared memory where it
@@ -25,9 +26,10 @@
 // GLA scales q and k around half the chunk's total per channel (exponents stay within half the total), and where a chunk's
 // total exceeds GLA_RANGE forms every score channel by channel instead (all exponents then <= 0). MLSTM needs no scaling of q
 // and k: with g_s = i_s - F_s and M_t = max(m_0, max_{s<=t} g_s), m_t = F_t + M_t, a score counts e^{g_s - M_t} and the old
-// state e^{m_0 - M_t}.
+// state e^{m_0 - M_t}. FIXED needs none of this: a score counts decay^(t - s), the old state decay^(t + 1), both as 2^ of the
+// head's binary logarithm.
 //
-// The products run on mma.sync (bf16 in, fp32 out). q, k and v of the MLSTM and v of the GLA are bfloat16 as projected; every
+// The products run on mma.sync (bf16 in, fp32 out). q, k and v of the MLSTM and of FIXED and v of the GLA are bfloat16 as projected; every
 // fp32 operand (scaled q and k, scores, the state) is carried as a sum of two bfloat16 values, which leaves a relative error
 // of about 2^-17 in it.
 #include "layout.cuh"
@@ -37,7 +39,7 @@ namespace {
 
 using namespace mmafrag;
 
-enum GmKind : int { GLA = 0, MLSTM = 1 };
+enum GmKind : int { GLA = 0, MLSTM = 1, FIXED = 2 };
 
 constexpr int GC = 64;                  // tokens of a chunk
 constexpr int G_THREADS = 256;
@@ -67,7 +69,7 @@ __device__ __forceinline__ float log2_sigmoid(float z) {
     return fminf(y, 0.f) - s;
 }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
-template <int KIND> __device__ __forceinline__ float gate_act(float z) { return KIND == GLA ? z * sigmoid_f(z) : sigmoid_f(z); }
+template <int KIND> __device__ __forceinline__ float gate_act(float z) { return KIND == MLSTM ? sigmoid_f(z) : z * sigmoid_f(z); }
 
 // ------------------------------------------------------------------------------------------------ token form
 constexpr int TOK_BATCH = 8;            // rows of S a thread has in flight
@@ -171,7 +173,7 @@ gm_token_kernel(const T* __restrict__ p, const T* __restrict__ w2, const float* 
                 }
                 as[c] = expf(log_sigmoid_f(z + (c == tid ? b_first : bias[h * dim + c])) * a.inv_tau);
             }
-        } else if (tid == 0) {
+        } else if (KIND == MLSTM && tid == 0) {
             const float i = a.cap * tanhf((to_f32(row[a.a_off + h]) + bias[h]) / a.cap);
             const float f = log_sigmoid_f(a.cap * tanhf((to_f32(row[a.b_off + h]) + bias[a.H + h]) / a.cap));
             const float m_new = fmaxf(f + m_s, i);
@@ -180,7 +182,7 @@ gm_token_kernel(const T* __restrict__ p, const T* __restrict__ w2, const float* 
             m_s = m_new;
         }
         __syncthreads();
-        const float keep = KIND == MLSTM ? keep_s : 0.f, add = KIND == MLSTM ? add_s : 1.f;
+        const float keep = KIND == MLSTM ? keep_s : (KIND == FIXED ? bias[h] : 0.f), add = KIND == MLSTM ? add_s : 1.f;
         float acc[VEC];
 #pragma unroll
         for (int j = 0; j < VEC; j++) acc[j] = 0.f;
@@ -457,7 +459,7 @@ gm_chunk_state_kernel(const bf16* __restrict__ p, const bf16* __restrict__ w2, c
             *reinterpret_cast<float4*>(zb + t * LZ + c) = v;
             if (t < nt) *reinterpret_cast<float4*>(sc.b + ((size_t)(t0 + t) * a.H + h) * dim + c) = v;
         }
-    } else {
+    } else if (KIND == MLSTM) {
         mlstm_gates(p, bias, t0, nt, h, a, zb, zb + GC, nullptr);
     }
     __syncthreads();
@@ -490,7 +492,7 @@ gm_chunk_state_kernel(const bf16* __restrict__ p, const bf16* __restrict__ w2, c
 #pragma unroll
                     for (int j = 0; j < 8; j++) kv[j] *= exp2f(be[j] - bt[j]);
                 } else {
-                    const float w = expf(zb[GC + t] - G);
+                    const float w = KIND == FIXED ? exp2f(bias[a.H + h] * (float)(nt - 1 - t)) : expf(zb[GC + t] - G);
 #pragma unroll
                     for (int j = 0; j < 8; j++) kv[j] *= w;
                 }
@@ -551,7 +553,7 @@ constexpr int SCAN_AHEAD = 4;           // chunks whose U is in flight
 // grid (groups of 4 * SCAN_THREADS entries of S, and behind them of n, H, B)
 template <int KIND>
 __global__ void __launch_bounds__(SCAN_THREADS)
-gm_chunk_scan_kernel(GmState st, GmScratch sc, const int* __restrict__ cu_q, const int* __restrict__ slots, GmArgs a) {
+gm_chunk_scan_kernel(GmState st, GmScratch sc, const float* __restrict__ bias, const int* __restrict__ cu_q, const int* __restrict__ slots, GmArgs a) {
     griddep_wait();
     const int h = blockIdx.y, b = blockIdx.z;
     const int slot = slots[b], q0 = cu_q[b], q1 = cu_q[b + 1];
@@ -577,6 +579,7 @@ gm_chunk_scan_kernel(GmState st, GmScratch sc, const int* __restrict__ cu_q, con
     };
     float4 S = live ? *reinterpret_cast<const float4*>(stp) : make_float4(0.f, 0.f, 0.f, 0.f);
     float m = KIND == MLSTM && live ? st.m[sh] : 0.f;
+    const float lg = KIND == FIXED ? bias[a.H + h] : 0.f;
     float4 u[SCAN_AHEAD], un[SCAN_AHEAD];
     float2 d[SCAN_AHEAD], dn[SCAN_AHEAD];
     auto fetch = [&](int c0, float4 (&uu)[SCAN_AHEAD], float2 (&dd)[SCAN_AHEAD]) {
@@ -586,6 +589,7 @@ gm_chunk_scan_kernel(GmState st, GmScratch sc, const int* __restrict__ cu_q, con
             if (c >= nch) continue;
             uu[i] = *u_of(c);
             if (KIND == GLA) dd[i].x = sc.b[((size_t)(min(q0 + (c + 1) * GC, q1) - 1) * a.H + h) * a.dim + row];
+            else if (KIND == FIXED) dd[i].x = lg * (float)(min(q0 + (c + 1) * GC, q1) - (q0 + c * GC));
             else dd[i] = *reinterpret_cast<const float2*>(sc.scal + ((size_t)(base + nch - 1 - c) * a.H + h) * 2);
         }
     };
@@ -598,7 +602,7 @@ gm_chunk_scan_kernel(GmState st, GmScratch sc, const int* __restrict__ cu_q, con
             if (c >= nch) continue;
             *u_of(c) = S;                                      // the state before the chunk
             float keep, add = 1.f;
-            if (KIND == GLA) {
+            if (KIND != MLSTM) {
                 keep = exp2f(d[i].x);
             } else {
                 if (e == 0) sc.m0[(size_t)(base + nch - 1 - c) * a.H + h] = m;
@@ -647,6 +651,7 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
     const bf16* prow = p + (size_t)t0 * a.ld;
     const size_t fh = (size_t)flat * a.H + h;
     float m0 = 0.f;
+    const float lg = KIND == FIXED ? bias[a.H + h] : 0.f;      // binary logarithm of the head's decay
     uint4 q_raw[4], k_raw[4];
     float4 b_raw[4][2];
     auto fetch_qkb = [&](const Pieces& pc) {
@@ -709,9 +714,11 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
         load_tile(qs, LK, prow + a.q_off + h * dim, a.ld, nt, dim, dimP);
         load_tile(ks, LK, prow + a.k_off + h * dim, a.ld, nt, dim, dimP);
         load_tile(vs, LV, prow + a.v_off + h * vd, a.ld, nt, vd, vdP);
-        m0 = sc.m0[fh];
-        mlstm_gates(p, bias, t0, nt, h, a, Fs, gs, Ms);
-        for (int c = tid; c < dimP; c += G_THREADS) rf[c] = c < dim ? sc.un[fh * dim + c] : 0.f;
+        if (KIND == MLSTM) {
+            m0 = sc.m0[fh];
+            mlstm_gates(p, bias, t0, nt, h, a, Fs, gs, Ms);
+            for (int c = tid; c < dimP; c += G_THREADS) rf[c] = c < dim ? sc.un[fh * dim + c] : 0.f;
+        }
         cp_async_wait<1>();                                    // q and k (the values land under the scores)
     }
     __syncthreads();
@@ -758,6 +765,9 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
                         x = key <= t ? x * a.q_scale * expf(gs[key] - Ms[t]) : 0.f;
                         y = key + 1 <= t ? y * a.q_scale * expf(gs[key + 1] - Ms[t]) : 0.f;
                         sum += x + y;
+                    } else if (KIND == FIXED) {
+                        x = key <= t ? x * a.q_scale * exp2f(lg * (float)(t - key)) : 0.f;
+                        y = key + 1 <= t ? y * a.q_scale * exp2f(lg * (float)(t - key - 1)) : 0.f;
                     }
                     float rx, ry;
                     *reinterpret_cast<uint32_t*>(As + t * LA + key) = hi_pack(x, y, rx, ry);
@@ -882,10 +892,12 @@ gm_chunk_out_kernel(const bf16* __restrict__ p, const float* __restrict__ bias, 
                         xn[j][e] = xm[j][e];
                     }
             }
-            if (KIND == MLSTM) {
+            if (KIND != GLA) {
 #pragma unroll
                 for (int mt = 0; mt < 4; mt++) {
-                    const float f0 = a.q_scale * expf(m0 - Ms[mt * 16 + g]), f1 = a.q_scale * expf(m0 - Ms[mt * 16 + g + 8]);
+                    const int ta = mt * 16 + g;
+                    const float f0 = a.q_scale * (KIND == FIXED ? exp2f(lg * (float)(ta + 1)) : expf(m0 - Ms[ta]));
+                    const float f1 = a.q_scale * (KIND == FIXED ? exp2f(lg * (float)(ta + 9)) : expf(m0 - Ms[ta + 8]));
 #pragma unroll
                     for (int j = 0; j < 2; j++) {
                         acc[ng][mt][j][0] *= f0; acc[ng][mt][j][1] *= f0;
@@ -1000,7 +1012,7 @@ int launch_chunks(const void* p, const void* w2, const float* bias, const float*
     mynah_launch(k1, dim3(chunks, a.H), dim3(G_THREADS), smem, stream, (const bf16*)p, (const bf16*)w2, bias, sc, cu_q, a);
     if (mynah_check_launch("gated_memory (chunk states)") != 0) return -1;
     const int entries = a.dim * a.vd / 4 + (KIND == MLSTM ? a.dim / 4 : 0);
-    mynah_launch(gm_chunk_scan_kernel<KIND>, dim3(ceil_div(entries, SCAN_THREADS), a.H, a.B), dim3(SCAN_THREADS), 0, stream, st, sc, cu_q, slots, a);
+    mynah_launch(gm_chunk_scan_kernel<KIND>, dim3(ceil_div(entries, SCAN_THREADS), a.H, a.B), dim3(SCAN_THREADS), 0, stream, st, sc, bias, cu_q, slots, a);
     if (mynah_check_launch("gated_memory (chunk scan)") != 0) return -1;
     constexpr int NQ = KIND == GLA ? 2 : 1;
     const size_t keys = (size_t)NQ * GC * (dimP + 8), scores = (size_t)2 * GC * (GC + 8);
@@ -1032,16 +1044,19 @@ static bool gm_chunked(int dtype, int dim, int vd, int rank, int max_q_len) {
 }
 
 // Floats of scratch that mynah_gated_memory wants for a step of `rows` rows in B sequences (0: it walks token by token).
-// kind 0: GLA, 1: MLSTM.
+// kind 0: GLA, 1: MLSTM, 2: FIXED.
 MYNAH_API long long mynah_gated_memory_scratch_floats(int kind, int dtype, int rows, int B, int H, int dim, int vd, int rank, int max_q_len) {
     if (!gm_chunked(dtype, dim, vd, rank, max_q_len)) return 0;
     const long long fh = (long long)(rows / GC + B) * H;
+    if (kind == FIXED) return fh * dim * vd;
     return kind == GLA ? fh * dim * vd + (long long)rows * H * dim : fh * ((long long)dim * vd + dim + 4);
 }
 
 // p: [rows][ld] rows whose columns hold, from q_off / k_off / v_off / g_off on, every head's q and k (dim values each), v and
 // gate (vd each); kind 0 (GLA): the narrow row of `rank` values at a_off, w2 [H * dim][rank] in dtype and bias fp32 [H * dim];
-// kind 1 (MLSTM): the heads' input gates at a_off and forget gates at b_off, bias fp32 [2 H] (input, then forget).
+// kind 1 (MLSTM): the heads' input gates at a_off and forget gates at b_off, bias fp32 [2 H] (input, then forget);
+// kind 2 (FIXED): bias fp32 [2 H], the heads' decays (not negative), then their binary logarithms (a finite number below -1e4
+// for a decay of zero).
 // w_norm: fp32 [H * vd]. State fp32: S [n_slots + 1][H][dim][vd]; kind 1 also n [...][dim] and m [...]. out: [rows][ldo] in
 // dtype. max_q_len: the most tokens a sequence brings. scratch: mynah_gated_memory_scratch_floats(...) floats, 16-byte aligned,
 // or null (token by token).
@@ -1051,9 +1066,9 @@ MYNAH_API int mynah_gated_memory(int kind, const void* p, int ld, int q_off, int
                                  const int* slots, int B, int rows, int H, int dim, int vd, int max_q_len, float* scratch,
                                  cudaStream_t stream) {
     if (B == 0 || rows == 0) return 0;
-    MYNAH_REQUIRE(kind == GLA || kind == MLSTM, "gated_memory: kind %d is neither 0 nor 1", kind);
+    MYNAH_REQUIRE(kind == GLA || kind == MLSTM || kind == FIXED, "gated_memory: kind %d is none of 0, 1, 2", kind);
     MYNAH_REQUIRE(B > 0 && rows > 0 && H > 0 && dim > 0 && vd > 0 && H <= 65535 && B <= 65535, "gated_memory: bad sizes");
-    MYNAH_REQUIRE(kind == GLA ? rank > 0 && w2 != nullptr : n != nullptr && m != nullptr && cap > 0.f, "gated_memory: what the kind needs is missing");
+    MYNAH_REQUIRE(bias != nullptr && (kind == FIXED || (kind == GLA ? rank > 0 && w2 != nullptr : n != nullptr && m != nullptr && cap > 0.f)), "gated_memory: what the kind needs is missing");
     MYNAH_REQUIRE(dtype == MYNAH_F32 || dtype == MYNAH_BF16, "gated_memory: unsupported dtype %d", dtype);
     const GmArgs a{B, H, dim, vd, ld, ldo, o_off, q_off, k_off, v_off, g_off, a_off, b_off, kind == GLA ? rank : 0, n_slots, q_scale, inv_tau, cap, eps};
     const GmState st{S, n, m};
@@ -1067,12 +1082,16 @@ MYNAH_API int mynah_gated_memory(int kind, const void* p, int ld, int q_off, int
             sc.b = scratch + fh * dim * vd;
             return launch_chunks<GLA>(p, w2, bias, w_norm, st, sc, out, cu_q, slots, a, rows, stream);
         }
+        if (kind == FIXED) return launch_chunks<FIXED>(p, w2, bias, w_norm, st, sc, out, cu_q, slots, a, rows, stream);
         sc.un = scratch + fh * dim * vd;
         sc.scal = sc.un + fh * dim;
         sc.m0 = sc.scal + 2 * fh;
         return launch_chunks<MLSTM>(p, w2, bias, w_norm, st, sc, out, cu_q, slots, a, rows, stream);
     }
-    MYNAH_REQUIRE(kind == MLSTM || dtype == MYNAH_F32 || ((uintptr_t)w2 & 15) == 0, "gated_memory: the narrow matrix is not aligned");
+    MYNAH_REQUIRE(kind != GLA || dtype == MYNAH_F32 || ((uintptr_t)w2 & 15) == 0, "gated_memory: the narrow matrix is not aligned");
+    if (kind == FIXED)
+        return dtype == MYNAH_F32 ? launch_token<float, FIXED>(p, w2, bias, w_norm, st, out, cu_q, slots, a, max_q_len, stream)
+                                  : launch_token<bf16, FIXED>(p, w2, bias, w_norm, st, out, cu_q, slots, a, max_q_len, stream);
     if (dtype == MYNAH_F32)
         return kind == GLA ? launch_token<float, GLA>(p, w2, bias, w_norm, st, out, cu_q, slots, a, max_q_len, stream)
                            : launch_token<float, MLSTM>(p, w2, bias, w_norm, st, out, cu_q, slots, a, max_q_len, stream);

@@ -39,7 +39,7 @@ constexpr int A_BYTES = BM * BK * 2;                 // 16 KB
 constexpr int THREADS = 192;
 constexpr int STAGING_BYTES = 32 * 128;              // 32 rows x 128 bytes per epilogue warp and buffer
 
-enum Epi : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_QKV = 3, EPI_GATED = 4, EPI_GELU = 5 };
+enum Epi : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_QKV = 3, EPI_GATED = 4, EPI_GELU = 5, EPI_RELU2 = 6 };
 
 // The two epilogues that read a gate tile and its up tile side by side: SwiGLU, and the clamped gate
 // g = min(gate, limit), u = clamp(up, -limit, limit), out = g * sigmoid(alpha g) * (u + 1).
@@ -115,6 +115,9 @@ struct GemmShape {
     const int* tile_group;
     int group_rows;
     float gate_limit, gate_alpha;   // of the clamped gate epilogue
+    // Of the squared relu: the accumulator of row r is multiplied by row_weight[row_pair[r]] first (row_pair -1: by zero); null: by 1
+    const int* row_pair;
+    const float* row_weight;
 };
 
 // What a unit works on next: a tile of C and a range of its k-blocks. Without SK that is a whole tile (or, with
@@ -428,6 +431,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             if (warp == 2 && lane == 0) GSTAMP(2, local, 0);
             const uint32_t t_row = tmem_base + buf * BN + ((uint32_t)(quad * 32) << 16);
             const int row0 = (m_tile * CTAS + rank) * BM + quad * 32;
+            float row_w = 1.0f;
+            if (EPI == EPI_RELU2 && g.row_pair != nullptr && row0 + lane < g.M) {
+                const int pr = g.row_pair[row0 + lane];
+                row_w = pr >= 0 ? g.row_weight[pr] : 0.f;
+            }
             if (SK && w.produce) {
                 // this CTA's part of a tile that the CTA before it owns: the accumulator goes to this CTA's slot
                 float* mine = g.sk_part + ((size_t)unit * BM + quad * 32 + lane) * BN;
@@ -583,7 +591,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                     for (int j = 0; j < 8; j++)
                         *reinterpret_cast<uint4*>(my_row + ((j ^ (lane & 7)) * 16)) = make_uint4(r[4 * j], r[4 * j + 1], r[4 * j + 2], r[4 * j + 3]);
-                } else if (EPI == EPI_BF16 || EPI == EPI_GELU) {
+                } else if (EPI == EPI_BF16 || EPI == EPI_GELU || EPI == EPI_RELU2) {
 #pragma unroll
                     for (int half = 0; half < 2; half++) {
                         uint32_t r[32];
@@ -595,6 +603,14 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                             for (int e = 0; e < 32; e++) {
                                 const float z = round_to<bf16>(__uint_as_float(r[e]));
                                 r[e] = __float_as_uint(0.5f * z * (1.0f + erff(z * 0.7071067811865476f)));
+                            }
+                        }
+                        if (EPI == EPI_RELU2) {
+                            // the weighted product rounded to bf16 first, as when it is stored before the activation
+#pragma unroll
+                            for (int e = 0; e < 32; e++) {
+                                const float z = fmaxf(round_to<bf16>(__uint_as_float(r[e]) * row_w), 0.f);
+                                r[e] = __float_as_uint(z * z);
                             }
                         }
 #pragma unroll
@@ -770,7 +786,8 @@ int sk_workspace(int n_ctas, float** part, int** flag) {
 template <int BN, int EPI, int CTAS, int KS = 1, bool SK = false>
 int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap& mc, int M, int N, int K, int up_offset,
                 int sm_count, int* status, cudaStream_t stream, const QkvEpilogue& qe = QkvEpilogue{},
-                const int* tile_group = nullptr, int group_rows = 0, float gate_limit = 0.f, float gate_alpha = 0.f) {
+                const int* tile_group = nullptr, int group_rows = 0, float gate_limit = 0.f, float gate_alpha = 0.f,
+                const int* row_pair = nullptr, const float* row_weight = nullptr) {
     constexpr int STAGES = ring_stages(BN, CTAS);
     constexpr size_t smem = (size_t)STAGES * (A_BYTES + BN * BK * 2 / CTAS) + 4 * 2 * STAGING_BYTES + 256 + 1024;
     auto kern = gemm_tcgen05_kernel<BN, EPI, CTAS, KS, SK>;
@@ -784,6 +801,7 @@ int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap&
     g.M = M; g.N = N; g.K = K; g.up_offset = up_offset;
     g.m_tiles = ceil_div(M, BM * CTAS);
     g.n_tiles = epi_glu(EPI) ? ceil_div(N, 128) : ceil_div(N, BN);
+    g.row_pair = row_pair; g.row_weight = row_weight;
     g.tile_group = tile_group; g.group_rows = group_rows; g.gate_limit = gate_limit; g.gate_alpha = gate_alpha;
     static_assert(CTAS == 1 || EPI != EPI_GATED, "the grouped products run on single CTAs");
     const long long tiles = (long long)g.m_tiles * g.n_tiles;
@@ -856,14 +874,15 @@ MYNAH_API int mynah_gemm_tcgen05_splits_k(int M, int N, int K, int sm_count) {
     return on && ceil_div(K, BK) >= 32 && (long long)ceil_div(M, BM) * ceil_div(N, 256) <= sm_count / 2;
 }
 
-// epilogue 0: C bf16 [M, N]; 1: C fp32 [M, N]; 2: SwiGLU, W holds N gate rows then N up rows, C bf16 [M, N].
+// epilogue 0: C bf16 [M, N]; 1: C fp32 [M, N]; 2: SwiGLU, W holds N gate rows then N up rows, C bf16 [M, N];
+// 6: relu(.)^2 of the product rounded to bf16, C bf16 [M, N].
 // A [M, K] and W [rows, K] are bf16, row-major, 16-byte aligned; ldc is C's row pitch in elements. `status`
 // receives MYNAH_ST_TIMEOUT if a wait inside the kernel ran out.
 MYNAH_API int mynah_gemm_tcgen05(const void* A, const void* W, void* C, int M, int N, int K, int ldc, int epilogue,
                                  int sm_count, int* status, cudaStream_t stream) {
     if (M == 0 || N == 0) return 0;
     MYNAH_REQUIRE(mynah_gemm_tcgen05_supported(M, N, K), "gemm_tcgen05: M=%d N=%d K=%d is not taken (N and K must be multiples of 8)", M, N, K);
-    MYNAH_REQUIRE(epilogue >= 0 && epilogue <= 2 && ldc >= N, "gemm_tcgen05: bad epilogue or output stride");
+    MYNAH_REQUIRE(((epilogue >= 0 && epilogue <= 2) || epilogue == EPI_RELU2) && ldc >= N, "gemm_tcgen05: bad epilogue or output stride");
     const int csize = epilogue == EPI_F32 ? 4 : 2;
     MYNAH_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0 && ((uintptr_t)C & 15) == 0 && (ldc * csize) % 16 == 0,
                   "gemm_tcgen05: operands must be 16-byte aligned and the output pitch a multiple of 16 bytes");
@@ -877,7 +896,7 @@ MYNAH_API int mynah_gemm_tcgen05(const void* A, const void* W, void* C, int M, i
     // The k-blocks of all tiles dealt out evenly (stream-K) where whole tiles would leave SMs idle in their last
     // wave and the k-blocks saved are worth more than the fix-up. MYNAH_GEMM_SK=0: never, 2: wherever it can run.
     static const int sk_mode = [] { const char* e = getenv("MYNAH_GEMM_SK"); return e == nullptr ? 1 : (e[0] == '0' ? 0 : (e[0] == '2' ? 2 : 1)); }();
-    if (epilogue != EPI_SWIGLU && !pair && sk_mode != 0) {
+    if (epilogue != EPI_SWIGLU && epilogue != EPI_RELU2 && !pair && sk_mode != 0) {
         const long long tiles_w = (long long)ceil_div(M, BM) * ceil_div(N, 256);
         const int nk = ceil_div(K, BK);
         const long long waves = (tiles_w + sm_count - 1) / sm_count;
@@ -922,6 +941,7 @@ MYNAH_API int mynah_gemm_tcgen05(const void* A, const void* W, void* C, int M, i
     (pair ? launch_gemm<BN_, EPI_, 2>(ma, mb, mc, M, N, K, epilogue == EPI_SWIGLU ? N : 0, sm_count, status, stream) \
           : launch_gemm<BN_, EPI_, 1>(ma, mb, mc, M, N, K, epilogue == EPI_SWIGLU ? N : 0, sm_count, status, stream))
     if (epilogue == EPI_SWIGLU) return MYNAH_GEMM_GO(256, EPI_SWIGLU);
+    if (epilogue == EPI_RELU2) return wide ? MYNAH_GEMM_GO(256, EPI_RELU2) : MYNAH_GEMM_GO(128, EPI_RELU2);
     if (epilogue == EPI_F32) return wide ? MYNAH_GEMM_GO(256, EPI_F32) : MYNAH_GEMM_GO(128, EPI_F32);
     return wide ? MYNAH_GEMM_GO(256, EPI_BF16) : MYNAH_GEMM_GO(128, EPI_BF16);
 #undef MYNAH_GEMM_GO
@@ -959,6 +979,26 @@ MYNAH_API int mynah_gemm_tcgen05_grouped(const void* A, const void* W, void* C, 
         return launch_gemm<256, EPI_SWIGLU, 1>(ma, mb, mc, M, N, K, N, sm_count, status, stream, QkvEpilogue{}, tile_group, group_rows);
     return launch_gemm<256, EPI_GATED, 1>(ma, mb, mc, M, N, K, N, sm_count, status, stream, QkvEpilogue{}, tile_group, group_rows,
                                           gate_limit, gate_alpha);
+}
+
+// The grouped product with the squared relu behind it: C = relu(w A . W^T)^2 in bf16, with w = pair_weight[row_pair[r]] for row r
+// of A (a row with row_pair -1 holds no token and gives zeros; row_pair null: w = 1 throughout).
+MYNAH_API int mynah_gemm_tcgen05_grouped_relu2(const void* A, const void* W, void* C, int M, int N, int K, int ldc, int groups, int group_rows,
+                                               const int* tile_group, const int* row_pair, const float* pair_weight, int sm_count, int* status,
+                                               cudaStream_t stream) {
+    if (M == 0 || N == 0) return 0;
+    MYNAH_REQUIRE(mynah_gemm_tcgen05_supported(M, N, K) && M % BM == 0 && ldc >= N, "gemm_tcgen05_grouped_relu2: M=%d N=%d K=%d is not taken", M, N, K);
+    MYNAH_REQUIRE(groups > 0 && tile_group != nullptr && group_rows >= N, "gemm_tcgen05_grouped_relu2: the matrices do not hold the product's rows");
+    MYNAH_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0 && ((uintptr_t)C & 15) == 0 && ldc % 8 == 0,
+                  "gemm_tcgen05_grouped_relu2: operands must be 16-byte aligned and the output pitch a multiple of 16 bytes");
+    MYNAH_REQUIRE(status != nullptr && (row_pair == nullptr || pair_weight != nullptr), "gemm_tcgen05_grouped_relu2: a status word is required, and weights with the rows' pairs");
+    if (sm_count <= 0) sm_count = mynah_sm_count();
+    CUtensorMap ma, mb, mc;
+    if (make_map(&ma, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, K, K, 128, BK)) return -1;
+    if (make_map(&mb, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (long long)groups * group_rows, K, K, 128, BK)) return -1;
+    if (make_map(&mc, C, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, N, ldc, 32, 64)) return -1;
+    return launch_gemm<256, EPI_RELU2, 1>(ma, mb, mc, M, N, K, 0, sm_count, status, stream, QkvEpilogue{}, tile_group, group_rows, 0.f, 0.f,
+                                          row_pair, pair_weight);
 }
 
 // The q/k/v projection of a prompt step with its epilogue: C = A . W^T as above (W rows: H heads of q, KV of k,

@@ -26,6 +26,11 @@
 //                 them are the token's experts, and each counts s (without the correction) times a constant.
 //                 Variants: scores softmax(W_r h) over all experts; a group counting its largest score; no correction.
 //                 A further row behind the router's matrix gives the gate of a shared expert: sigmoid of its product.
+//   act: relu2    y = relu(W_up,e h)^2, one matrix an expert, no gate
+//   weight on the input   an expert reads weight_pair * h instead of h, and its rows are summed as they are. The products of
+//                 the expert's first matrices are linear in h, so the weight multiplies their fp32 accumulators.
+//   shared as an expert   a shared expert of the experts' own size can lie behind them in the stacked matrices: every token then
+//                 has one more pair, of expert number E and weight 1 (no gate), and needs no products of its own
 //   shared expert   a feed-forward that every token passes: its rows, made by the ordinary products, join in moe_combine
 //                 times the token's gate
 //   clamped gate    with limit = infinity, alpha = 1 and shift 0 it is the plain silu(g) * u
@@ -92,14 +97,22 @@ moe_route_kernel(const int* __restrict__ tokens, const int* __restrict__ tok_seq
     }
 }
 
-enum MoeAct : int { MOE_ACT_CLAMPED_GATE = 0, MOE_ACT_GELU = 1 };
+enum MoeAct : int { MOE_ACT_CLAMPED_GATE = 0, MOE_ACT_GELU = 1, MOE_ACT_RELU2 = 2 };
 
 struct MoeArgs {
     int top, D, F;
     float limit, alpha, shift;        // y = g sigmoid(alpha g) (u + shift), g and u clamped by limit
+    const float* in_weight;           // null, or the pair's weight on the expert's input [P]
+    __device__ __forceinline__ float weight_of(int p) const { return in_weight != nullptr ? in_weight[p] : 1.0f; }
 };
 
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+// the experts with one matrix before the activation
+template <int ACT> __device__ __forceinline__ float plain_act(float z) {
+    if (ACT == MOE_ACT_GELU) return gelu_erf_f(z);
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+}
 
 // grid (tiles, column tiles of F). h: [T][D] rows; w_gu: [E][2][F][D] (gate rows, then up rows); y: [P][F]
 template <typename TA, int BM, int ACT>
@@ -128,17 +141,18 @@ moe_gate_up_kernel(const TA* __restrict__ h, const TA* __restrict__ w_gu, TA* __
     for (int i = 0; i < BM / 16; i++) {
         const int p = pair_s[ty + 16 * i];
         if (p < 0) continue;
+        const float wt = a.weight_of(p);
 #pragma unroll
         for (int j = 0; j < BN / 16; j++) {
             const int c = c0 + tx + 16 * j;
             if (c >= a.F) continue;
             // the products are rounded to the activation type first, as a product kernel would store them
-            if (ACT == MOE_ACT_GELU) {
-                y[(size_t)p * a.F + c] = from_f32<TA>(gelu_erf_f(round_to<TA>(g[i][j])));
+            if (ACT != MOE_ACT_CLAMPED_GATE) {
+                y[(size_t)p * a.F + c] = from_f32<TA>(plain_act<ACT>(round_to<TA>(g[i][j] * wt)));
                 continue;
             }
-            const float gv = fminf(round_to<TA>(g[i][j]), a.limit);
-            const float uv = fminf(fmaxf(round_to<TA>(u[i][j]), -a.limit), a.limit);
+            const float gv = fminf(round_to<TA>(g[i][j] * wt), a.limit);
+            const float uv = fminf(fmaxf(round_to<TA>(u[i][j] * wt), -a.limit), a.limit);
             y[(size_t)p * a.F + c] = from_f32<TA>(gv * (1.0f / (1.0f + expf(-a.alpha * gv))) * (uv + a.shift));
         }
     }
@@ -185,7 +199,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ o, const int* __res
     griddep_launch_small();
     griddep_wait();
     const int t = blockIdx.x;
-    const float sg = shared != nullptr ? shared_gate[t] : 0.f;
+    const float sg = shared != nullptr ? (shared_gate != nullptr ? shared_gate[t] : 1.0f) : 0.f;
     if (D % 4 == 0) {                                       // four columns a thread, 16-byte loads; a column's sum runs in the same order
         for (int c = threadIdx.x * 4; c < D; c += blockDim.x * 4) {
             float acc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -314,14 +328,14 @@ template <typename TA>
 __global__ void __launch_bounds__(ROUTER_THREADS)
 moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecRef correction, const int* __restrict__ tok_seq,
                         int* __restrict__ choice, float* __restrict__ pair_weight, float* __restrict__ shared_gate, int D, int E,
-                        int top, int groups, int keep, float weight_scale, int softmax_scores, int group_max) {
+                        int top, int groups, int keep, float weight_scale, int softmax_scores, int group_max, int extra) {
     __shared__ float sc[MOE_MAX_EXPERTS], ch[MOE_MAX_EXPERTS], gs[MOE_MAX_EXPERTS];
     griddep_wait();
-    const int t = blockIdx.x;
+    const int t = blockIdx.x, ld = top + extra;             // extra 1: a last pair of expert E and weight 1 (the shared expert)
     if (tok_seq[t] < 0) {
-        for (int k = threadIdx.x; k < top; k += blockDim.x) {
-            choice[t * top + k] = -1;
-            pair_weight[t * top + k] = 0.f;
+        for (int k = threadIdx.x; k < ld; k += blockDim.x) {
+            choice[t * ld + k] = -1;
+            pair_weight[t * ld + k] = 0.f;
         }
         if (shared_gate != nullptr && threadIdx.x == 0) shared_gate[t] = 0.f;
         return;
@@ -414,11 +428,15 @@ moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecR
             if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
         }
         if (lane == 0) {
-            choice[t * top + k] = at < E ? at : -1;
-            pair_weight[t * top + k] = at < E ? sc[at] * weight_scale : 0.f;
+            choice[t * ld + k] = at < E ? at : -1;
+            pair_weight[t * ld + k] = at < E ? sc[at] * weight_scale : 0.f;
             if (at < E) ch[at] = -INFINITY;
         }
         __syncwarp();
+    }
+    if (extra && lane == 0) {
+        choice[t * ld + top] = E;
+        pair_weight[t * ld + top] = 1.0f;
     }
 }
 
@@ -456,18 +474,19 @@ moe_gate_up_mma_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w_gu
         for (int half = 0; half < 2; half++) {
             const int p = pair_s[m * 16 + g + 8 * half];
             if (p < 0) continue;
+            const float wt = a.weight_of(p);
 #pragma unroll
             for (int j = 0; j < NT; j++)
 #pragma unroll
                 for (int q = 0; q < 2; q++) {
                     const int c = c0 + j * 8 + 2 * t + q;
                     if (c >= a.F) continue;
-                    if (ACT == MOE_ACT_GELU) {
-                        y[(size_t)p * a.F + c] = from_f32<bf16>(gelu_erf_f(round_to<bf16>(acc[0][m][j][2 * half + q])));
+                    if (ACT != MOE_ACT_CLAMPED_GATE) {
+                        y[(size_t)p * a.F + c] = from_f32<bf16>(plain_act<ACT>(round_to<bf16>(acc[0][m][j][2 * half + q] * wt)));
                         continue;
                     }
-                    const float gv = fminf(round_to<bf16>(acc[0][m][j][2 * half + q]), a.limit);
-                    const float uv = fminf(fmaxf(round_to<bf16>(acc[NMAT - 1][m][j][2 * half + q]), -a.limit), a.limit);
+                    const float gv = fminf(round_to<bf16>(acc[0][m][j][2 * half + q] * wt), a.limit);
+                    const float uv = fminf(fmaxf(round_to<bf16>(acc[NMAT - 1][m][j][2 * half + q] * wt), -a.limit), a.limit);
                     y[(size_t)p * a.F + c] = from_f32<bf16>(gv * (1.0f / (1.0f + expf(-a.alpha * gv))) * (uv + a.shift));
                 }
         }
@@ -619,6 +638,9 @@ MYNAH_API int mynah_moe_grouped_min(int n) {
 extern "C" int mynah_gemm_tcgen05_grouped(const void* A, const void* W, void* C, int M, int N, int K, int ldc, int epilogue, int groups,
                                int group_rows, const int* tile_group, float gate_limit, float gate_alpha, int sm_count,
                                int* status, cudaStream_t stream);
+extern "C" int mynah_gemm_tcgen05_grouped_relu2(const void* A, const void* W, void* C, int M, int N, int K, int ldc, int groups, int group_rows,
+                                                const int* tile_group, const int* row_pair, const float* pair_weight, int sm_count, int* status,
+                                                cudaStream_t stream);
 
 // Rows of the sorted, padded layout of a step whose products run grouped; 0: the step runs tile by tile instead.
 MYNAH_API int mynah_moe_grouped_rows(int T, int top, int E, int D, int F, int dtype) {
@@ -639,7 +661,9 @@ static int moe_run(const void* h, int dtype, const int* tokens, const int* tok_s
                    const float* pair_weight, const void* w_gu, const void* w_down, void* out, int out_f32, void* y, float* o,
                    int* ints, void* a_sorted, int T, int V, int top, int E, int D, int F, int act, float limit, float alpha,
                    float weight, int* status, cudaStream_t stream, float shift = 1.0f, const float* shared = nullptr,
-                   const float* shared_gate = nullptr) {
+                   const float* shared_gate = nullptr, int on_input = 0) {
+    const float* in_weight = on_input ? pair_weight : nullptr;      // on the experts' inputs: the sum then takes their rows as they are
+    if (on_input) { pair_weight = nullptr; weight = 1.0f; }
     const int P = T * top, BM = mynah_moe_tile_rows(T, top), max_tiles = mynah_moe_max_tiles(T, top, E);
     int* pair_expert = ints;
     int* perm = ints + P;
@@ -655,7 +679,9 @@ static int moe_run(const void* h, int dtype, const int* tokens, const int* tok_s
         if (mynah_check_launch("moe_route") != 0) return -1;
         mynah_launch(moe_gather_kernel, dim3(m_pad), dim3(128), 0, stream, (const bf16*)h, (const int*)perm_pad, (bf16*)a_sorted, top, D);
         if (mynah_check_launch("moe_gather") != 0) return -1;
-        if (act == MOE_ACT_GELU) {
+        if (act == MOE_ACT_RELU2) {
+            if (mynah_gemm_tcgen05_grouped_relu2(a_sorted, w_gu, y, m_pad, F, D, F, E, F, tile_group, in_weight != nullptr ? perm_pad : nullptr, in_weight, 0, status, stream) != 0) return -1;
+        } else if (act == MOE_ACT_GELU) {
             if (mynah_gemm_tcgen05_grouped(a_sorted, w_gu, y, m_pad, F, D, F, 5, E, F, tile_group, 0.f, 0.f, 0, status, stream) != 0) return -1;
         } else {
             // shift 1: the clamped gate; shift 0 (then limit is infinite and alpha 1): the plain silu gate, an epilogue of its own
@@ -673,7 +699,7 @@ static int moe_run(const void* h, int dtype, const int* tokens, const int* tok_s
     mynah_launch(moe_route_kernel, dim3(1), dim3(MOE_ROUTE_THREADS), 0, stream, tokens, tok_seq, table, choice, T, V, top, E, BM,
                  pair_expert, perm, tiles, max_tiles, status);
     if (mynah_check_launch("moe_route") != 0) return -1;
-    const MoeArgs a{top, D, F, limit, alpha, shift};
+    const MoeArgs a{top, D, F, limit, alpha, shift, in_weight};
     int rc;
     // bfloat16 rows that can move 16 bytes at a time take the tensor-core kernels
     const bool mma_ok = dtype == MYNAH_BF16 && D % 8 == 0 && F % 8 == 0 && !g_moe_plain &&
@@ -689,6 +715,7 @@ static int moe_run(const void* h, int dtype, const int* tokens, const int* tok_s
         rc = BM == 16 ? launch_products<bf16, 16, ACT_>(h, w_gu, w_down, y, o, perm, tiles, max_tiles, a, stream)      \
                       : launch_products<bf16, 64, ACT_>(h, w_gu, w_down, y, o, perm, tiles, max_tiles, a, stream)
     if (act == MOE_ACT_GELU) { MOE_GO(MOE_ACT_GELU); }
+    else if (act == MOE_ACT_RELU2) { MOE_GO(MOE_ACT_RELU2); }
     else { MOE_GO(MOE_ACT_CLAMPED_GATE); }
 #undef MOE_GO
     if (rc != 0) return rc;
@@ -747,11 +774,15 @@ MYNAH_API int mynah_moe_router_ffn(const void* h, int dtype, const int* tok_seq,
 // shared expert, added times shared_gate [T], which the router writes from a further row of w_router ([E + 1][D]).
 // w_router [E][D] in dtype, correction [E] in c_dtype (or null); w_gu [E][2][F][D]; w_down [E][D][F];
 // out [T][D] in the activation type, or fp32 when out_f32. Scratch as for the learned router.
+// act MOE_ACT_RELU2: the experts are W_down relu(W_up h)^2, w_gu [E][F][D] (limit, alpha and shift are not read). on_input: a pair's
+// weight multiplies its expert's input instead of its output (one-matrix experts). extra 1: expert number E of the stacked
+// matrices is a shared expert that every token passes with weight 1; choice, pair_weight and the scratch then have top + 1 pairs
+// a token. shared_gate null: the rows `shared` are added as they are.
 MYNAH_API int mynah_moe_group_router_ffn(const void* h, int dtype, const int* tok_seq, const void* w_router, const void* correction,
                                          int c_dtype, const void* w_gu, const void* w_down, void* out, int out_f32, void* y, float* o,
                                          int* ints, void* a_sorted, int* choice, float* pair_weight, int T, int top, int E, int D,
                                          int F, int groups, int keep, float weight_scale, int softmax_scores, int group_max, float limit,
-                                         float alpha, float shift, const float* shared, float* shared_gate, int* status,
+                                         float alpha, float shift, const float* shared, float* shared_gate, int act, int on_input, int extra, int* status,
                                          cudaStream_t stream) {
     if (T == 0) return 0;
     MYNAH_REQUIRE(T > 0 && top > 0 && E > 0 && top <= E && D > 0 && F > 0, "moe_group_router_ffn: bad sizes");
@@ -759,17 +790,19 @@ MYNAH_API int mynah_moe_group_router_ffn(const void* h, int dtype, const int* to
     MYNAH_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups, "moe_group_router_ffn: %d experts do not form %d groups of which %d are kept", E, groups, keep);
     MYNAH_REQUIRE(top <= keep * (E / groups), "moe_group_router_ffn: %d experts a token exceed those of %d kept groups", top, keep);
     MYNAH_REQUIRE(shift == 1.0f || (shift == 0.f && limit > 3.0e38f && alpha == 1.0f), "moe_group_router_ffn: the experts' gate is the clamped one (shift 1) or the plain silu (shift 0, no limit, alpha 1)");
-    MYNAH_REQUIRE(shared == nullptr || shared_gate != nullptr, "moe_group_router_ffn: a shared expert's rows need its gates");
+    MYNAH_REQUIRE(act == MOE_ACT_CLAMPED_GATE || act == MOE_ACT_RELU2, "moe_group_router_ffn: activation %d is not built in", act);
+    MYNAH_REQUIRE(!on_input || act == MOE_ACT_RELU2, "moe_group_router_ffn: a weight on the input goes with the one-matrix experts");
+    MYNAH_REQUIRE(extra == 0 || (extra == 1 && shared == nullptr && on_input && E < MOE_MAX_EXPERTS), "moe_group_router_ffn: a shared expert in the stack goes with weights on the input and without rows of its own");
     const VecRef corr{correction, c_dtype};
     if (dtype == MYNAH_F32)
         mynah_launch(moe_group_router_kernel<float>, dim3(T), dim3(router_threads(T, E)), 0, stream, (const float*)h, (const float*)w_router,
-                     corr, tok_seq, choice, pair_weight, shared_gate, D, E, top, groups, keep, weight_scale, softmax_scores, group_max);
+                     corr, tok_seq, choice, pair_weight, shared_gate, D, E, top, groups, keep, weight_scale, softmax_scores, group_max, extra);
     else if (dtype == MYNAH_BF16)
         mynah_launch(moe_group_router_kernel<bf16>, dim3(T), dim3(router_threads(T, E)), 0, stream, (const bf16*)h, (const bf16*)w_router,
-                     corr, tok_seq, choice, pair_weight, shared_gate, D, E, top, groups, keep, weight_scale, softmax_scores, group_max);
+                     corr, tok_seq, choice, pair_weight, shared_gate, D, E, top, groups, keep, weight_scale, softmax_scores, group_max, extra);
     else
         return mynah_fail("moe_group_router_ffn: unsupported dtype %d", dtype);
     if (mynah_check_launch("moe_group_router") != 0) return -1;
     return moe_run(h, dtype, nullptr, tok_seq, nullptr, choice, pair_weight, w_gu, w_down, out, out_f32, y, o, ints, a_sorted, T, 1,
-                   top, E, D, F, MOE_ACT_CLAMPED_GATE, limit, alpha, 1.0f, status, stream, shift, shared, shared_gate);
+                   top + extra, E + extra, D, F, act, limit, alpha, 1.0f, status, stream, shift, shared, shared_gate, on_input);
 }

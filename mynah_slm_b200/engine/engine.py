@@ -229,6 +229,9 @@ class Engine:
             fill_into(self.model.tensor_specs(), checkpoint, self.runtime)
         else:
             load_into(self.model.tensor_specs(), checkpoint, self.runtime)
+        for part in self.model.parts():            # parts without tensors learn of the run as well
+            if not part.tensor_specs():
+                part.bind({}, self.runtime)
         self.max_seqs = int(max_seqs) if max_seqs else min(self.n_pages, 1024)
         self.cache = Cache(self.model.cache_plan(), self.n_pages, self.max_seqs, dtype, self.device)
         self.n_groups = len(self.cache.plan.groups)
@@ -357,6 +360,7 @@ class Engine:
                 stream.add_f32(x0)
             if e.add_vector is not None:
                 kernels.residual_add_row(stream.flush(), self.model.stream_vectors.rows[e.add_vector])
+                stream.rounded = None
             self.model.layers[e.layer].forward(stream, ctx, views[i])
             if taps is not None:
                 taps[f"layer{i}"] = stream.flush().clone()
@@ -510,10 +514,13 @@ class Engine:
                 stream.add_f32(x0)
             if e.add_vector is not None:
                 kernels.residual_add_row(stream.flush(), self.model.stream_vectors.rows[e.add_vector])
+                stream.rounded = None
             self.model.layers[e.layer].forward(stream, ctx, self.cache.views[i])
 
     def _embed(self, ctx: StepContext) -> torch.Tensor:
         emb = self.model.embedding
+        if self.cache.embedding_state is not None:     # one that keeps something of every sequence from step to step
+            return emb.forward(ctx.tokens, ctx, self.cache.embedding_state)
         if getattr(emb, "needs_context", False):       # an embedding that also reads the rows' positions
             return emb.forward(ctx.tokens, ctx)
         return emb.forward(ctx.tokens)

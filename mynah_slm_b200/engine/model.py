@@ -7,7 +7,7 @@ cache and sorts the runs into storage groups.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Optional
 
 import torch
@@ -33,6 +33,7 @@ class EntryPlan:
 class CachePlan:
     groups: list[GroupPlan] = field(default_factory=list)
     entries: list[EntryPlan] = field(default_factory=list)
+    embedding_state: object = None       # a StateRequest of the model's embedding
 
 
 class Model:
@@ -67,15 +68,23 @@ class Model:
         return [(p, ts) for p in self.parts() for ts in p.tensor_specs()]
 
     def cache_plan(self) -> CachePlan:
-        plan = CachePlan()
+        plan = CachePlan(embedding_state=self.embedding.state_request())
         keys: dict[tuple, int] = {}
+        # how far back an entry's cache must reach: as far as it or any entry that reads it looks (None: everywhere)
+        reach: dict[int, Optional[int]] = {}
+        for i, e in enumerate(self.schedule):
+            kv = self.layers[e.layer].mixer.kv_request()
+            if kv is not None:
+                src = i if e.cache_from is None else e.cache_from
+                have = reach.get(src, 0)
+                reach[src] = None if kv.window is None or have is None else max(have, kv.window)
         for i, e in enumerate(self.schedule):
             mixer = self.layers[e.layer].mixer
             kv, st = mixer.kv_request(), mixer.state_request()
             if e.cache_from is not None:
                 src = self.schedule[e.cache_from]
                 src_kv = self.layers[src.layer].mixer.kv_request()
-                if kv is None or src_kv != kv:
+                if kv is None or src_kv is None or replace(src_kv, window=kv.window) != kv:
                     raise ConfigError(f"schedule[{i}] reads the cache of entry {e.cache_from}, "
                                       f"but asks for {kv} where that entry keeps {src_kv}")
                 if st is not None:
@@ -84,10 +93,10 @@ class Model:
                 continue
             ep = EntryPlan(state=st, block_state=self.layers[e.layer].state_request())
             if kv is not None:
-                key = (kv.kv_heads, kv.head_dim, kv.window, kv.value_dim, kv.value_heads)
+                key = (kv.kv_heads, kv.head_dim, reach[i], kv.value_dim, kv.value_heads)
                 if key not in keys:
                     keys[key] = len(plan.groups)
-                    plan.groups.append(GroupPlan(kv.kv_heads, kv.head_dim, kv.window, v_head_dim=kv.value_dim,
+                    plan.groups.append(GroupPlan(kv.kv_heads, kv.head_dim, reach[i], v_head_dim=kv.value_dim,
                                                  v_heads=kv.value_heads))
                 g = keys[key]
                 ep.group, ep.index_in_group = g, len(plan.groups[g].entries)

@@ -118,39 +118,39 @@ def _tc_capped_fits(HD: int, VD: int, scale: float, softcap: float, vdo: int) ->
 
 def prefill_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int, k_cache, v_cache, pages,
                    window: int, scale: float, softcap: float, keep_first: int, vdiv: int, null_key: bool = False,
-                   out_scale: float = 1.0, vdo=None) -> None:
+                   out_scale: float = 1.0, vdo=None, sink=None) -> None:
     """Prompt attention for mixers whose scores are capped, whose window keeps a sequence's first tokens, whose key heads
-    share value heads (`vdiv` key heads a value head), whose softmax holds one more term of score 0 without a value
-    (`null_key`), whose output carries a factor, or whose output heads are narrower (`vdo` columns) than the stored value
+    share value heads (`vdiv` key heads a value head), whose softmax holds one more term without a value, of score 0
+    (`null_key`) or of a score of its own for every query head (`sink`), whose output carries a factor, or whose output heads are narrower (`vdo` columns) than the stored value
     heads. Without any of these it is `prefill_masked`; the tcgen05 kernel takes bfloat16 heads of 64 or 128, the general
     kernel the rest."""
     vdo = VD if vdo is None else int(vdo)
-    plain = not null_key and out_scale == 1.0 and vdo == VD
+    plain = not null_key and sink is None and out_scale == 1.0 and vdo == VD
     if plain and not softcap and not keep_first and vdiv == 1 and out.is_contiguous():
         prefill_masked(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, 0, scale)
         return
     if (USE_TCGEN05_PREFILL and _tc_capped_fits(HD, VD, scale, softcap, vdo)
             and kernels.attn_prefill_tcgen05_supported(q.dtype, H, KV, HD)):
         kernels.attn_prefill_tcgen05_capped(q, out, ctx, H, KV, HD, k_cache, v_cache, pages, window, scale, softcap,
-                                            keep_first, vdiv, VD, null_key, out_scale, vdo)
+                                            keep_first, vdiv, VD, null_key, out_scale, vdo, sink)
         return
     kernels.attn_prefill_capped(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, scale, softcap, keep_first, vdiv,
-                                null_key, out_scale, vdo)
+                                null_key, out_scale, vdo, sink)
 
 
 def decode_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int, k_cache, v_cache, pages,
                   window: int, scale: float, softcap: float, keep_first: int, vdiv: int, scratch: torch.Tensor,
-                  null_key: bool = False, out_scale: float = 1.0, vdo=None) -> None:
+                  null_key: bool = False, out_scale: float = 1.0, vdo=None, sink=None) -> None:
     """The same choice for a decode step."""
     vdo = VD if vdo is None else int(vdo)
-    plain = not null_key and out_scale == 1.0 and vdo == VD
+    plain = not null_key and sink is None and out_scale == 1.0 and vdo == VD
     if plain and not softcap and not keep_first and vdiv == 1 and out.is_contiguous():
         decode_masked(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, 0, scale, scratch)
         return
     if (_tc_capped_fits(HD, VD, scale, softcap, vdo) and kernels.attn_decode_tc_supported(q.dtype, H, KV, HD)
             and _tc_fits(H, KV, ctx.decode_splits)):
         kernels.attn_decode_tc_capped(q, out, ctx, H, KV, HD, k_cache, v_cache, pages, window, scale, softcap, keep_first,
-                                      vdiv, scratch, VD, null_key, out_scale, vdo)
+                                      vdiv, scratch, VD, null_key, out_scale, vdo, sink)
         return
     kernels.attn_decode_capped(q, out, ctx, H, KV, HD, VD, k_cache, v_cache, pages, window, scale, softcap, keep_first, vdiv,
-                               scratch, null_key, out_scale, vdo)
+                               scratch, null_key, out_scale, vdo, sink)

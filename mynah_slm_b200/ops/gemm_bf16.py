@@ -59,7 +59,7 @@ def splits_k(M: int, N: int, K: int, device) -> bool:
 
 
 def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, N: int, epilogue: int, out: torch.Tensor) -> torch.Tensor:
-    """epilogue 0: bf16 rows, 1: fp32 rows, 2: SwiGLU (w = N gate rows then N up rows)."""
+    """epilogue 0: bf16 rows, 1: fp32 rows, 2: SwiGLU (w = N gate rows then N up rows), 6: relu(.)^2."""
     M, K = x.shape
     call("mynah_gemm_tcgen05", ptr(x), ptr(w), ptr(out), M, N, K, out.shape[1], epilogue, _sm_count(x.device),
          ptr(status_word(x.device)), stream_ptr())

@@ -56,6 +56,23 @@ def embed_gather(table: torch.Tensor, tokens: torch.Tensor, out: Optional[torch.
     return out
 
 
+def embed_pairs(table: torch.Tensor, pairs: torch.Tensor, last_token: torch.Tensor, ctx, mul_prev: int, mul_cur: int) -> torch.Tensor:
+    """x[t] = table[token_t] + pairs[row_t], fp32 [T, D]: row_t = (token before * mul_prev + token_t * mul_cur) mod buckets, the
+    last row of `pairs` for a sequence's first token. last_token int32 [slots + 1]: every sequence's last token, read for the
+    first row of its piece and left behind for its next step (csrc/elementwise.cu)."""
+    _chk(table, "embedding table", dim=2)
+    _chk(pairs, "pair table", table.dtype, 2)
+    _chk(last_token, "last tokens", torch.int32, 1)
+    T, (V, D) = ctx.tokens.numel(), table.shape
+    if pairs.shape[1] != D or pairs.shape[0] < 2:
+        raise KernelError("embed_pairs: the pair table does not fit the embedding")
+    out = torch.empty((T, D), dtype=torch.float32, device=table.device)
+    call("mynah_embed_pairs", ptr(table), ptr(pairs), code(table.dtype), ptr(ctx.tokens), ptr(ctx.tok_seq), ptr(ctx.tok_pos), ptr(ctx.cu_q),
+         ptr(ctx.slots), ptr(last_token), ptr(out), T, D, V, last_token.numel() - 1, pairs.shape[0] - 1, int(mul_prev), int(mul_cur),
+         ptr(ctx.status), stream_ptr())
+    return out
+
+
 def rmsnorm(x: torch.Tensor, gain: torch.Tensor, eps: float, act_dtype: torch.dtype,
             delta: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
             out: Optional[torch.Tensor] = None, delta_scale: float = 1.0) -> torch.Tensor:
@@ -268,6 +285,19 @@ def linear_swiglu(x, w_gate_up: torch.Tensor) -> torch.Tensor:
         gemm_bf16.counters["own"] += 1
         return gemm_bf16.gemm_tcgen05(x, w_gate_up, F, 2, out)      # the activation runs on the accumulator
     return swiglu(linear(x, w_gate_up))
+
+
+def linear_relu2(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """relu(x . w^T)^2 in x's type; one kernel for many bf16 rows (the activation runs on the accumulator)."""
+    from . import gemm_bf16
+    N = w.shape[0]
+    if (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and gemm_bf16.USE_TCGEN05 and x.shape[0] >= gemm_bf16.TCGEN05_MIN_ROWS
+            and x.is_contiguous() and w.is_contiguous() and gemm_bf16.tcgen05_supported(x.shape[0], N, x.shape[1])):
+        out = torch.empty((x.shape[0], N), dtype=torch.bfloat16, device=x.device)
+        gemm_bf16.counters["own"] += 1
+        return gemm_bf16.gemm_tcgen05(x, w, N, 6, out)
+    u = linear(x, w)
+    return activation(u, "relu2", out=u)
 
 
 def rope_table(n_pos: int, rotary_dim: int, theta: float, device) -> tuple[torch.Tensor, torch.Tensor]:
@@ -635,11 +665,13 @@ def causal_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], 
 
 def attn_prep(qkv: torch.Tensor, q_out: torch.Tensor, H: int, G: int, dim: int, vd: int, dimp: int, vdp: int,
               q_gain: torch.Tensor, k_gain: torch.Tensor, eps: float, cos, sin, rot: int, ctx, pages: PageTableView,
-              k_cache, v_cache, v_first: Optional[torch.Tensor], lam: Optional[torch.Tensor], vmix: int) -> None:
-    """Whole-projection q/k norm, partial rotation, per-head value norm, value mixing, cache write (csrc/attn_prep.cu)."""
+              k_cache, v_cache, v_first: Optional[torch.Tensor], lam: Optional[torch.Tensor], vmix: int,
+              value_norm: bool = True) -> None:
+    """Whole-projection q/k norm, partial rotation, per-head value norm (optional), value mixing, cache write
+    (csrc/attn_prep.cu)."""
     _chk(qkv, "qkv", dim=2)
     _chk(q_out, "q", qkv.dtype, 2)
-    if q_gain.dtype != k_gain.dtype or q_gain.numel() != H * dim or k_gain.numel() != G * dim:
+    if q_gain.dtype != k_gain.dtype or q_gain.numel() != H * dim or (k_cache is not None and k_gain.numel() != G * dim):
         raise KernelError("attn_prep: the gains must cover the whole q and k projections, in one dtype")
     if k_cache is not None:
         if k_cache.dtype != qkv.dtype or v_cache.dtype != qkv.dtype:
@@ -659,7 +691,7 @@ def attn_prep(qkv: torch.Tensor, q_out: torch.Tensor, H: int, G: int, dim: int, 
          H, G, dim, vd, dimp, vdp, ptr(q_gain), ptr(k_gain), code(q_gain.dtype), float(eps),
          ptr(cos), ptr(sin), rot, n_pos, ptr(ctx.tok_seq), ptr(ctx.tok_pos),
          ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages,
-         ptr(k_cache), ptr(v_cache), ptr(v_first), ptr(lam), vmix, ptr(ctx.status), stream_ptr())
+         ptr(k_cache), ptr(v_cache), ptr(v_first), ptr(lam), vmix, 1 if value_norm else 0, ptr(ctx.status), stream_ptr())
 
 
 def attn_prefill_general(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int,
@@ -884,11 +916,11 @@ def latent_prep(q: torch.Tensor, q_off: int, dkv: Optional[torch.Tensor], dkv_of
 
 
 def head_linear(x: torch.Tensor, head_in: int, in_off: int, W: torch.Tensor, out: torch.Tensor, head_out: int,
-                out_off: int, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                out_off: int, gate: Optional[torch.Tensor] = None, gate_cols: bool = False) -> torch.Tensor:
     """out[t, h * head_out + out_off + j] = sum_i W[h, j, i] * x[t, h * head_in + in_off + i]: one small product a head
     (csrc/latent_attn.cu). W [H, n_out, n_in] in the rows' type; fp32 accumulation. With `gate` (rows of H logits in
     the rows' type; a column slice is fine) head h's outputs are multiplied by sigmoid(gate[t, h]) before they are
-    rounded."""
+    rounded; with gate_cols the gate has a column for every output, gate[t, h * n_out + j]."""
     _rows(x, "head_linear: input")
     _rows(out, "head_linear: output")
     _chk(W, "head_linear: weights", x.dtype, 3)
@@ -899,11 +931,11 @@ def head_linear(x: torch.Tensor, head_in: int, in_off: int, W: torch.Tensor, out
         raise KernelError("head_linear: the heads do not fit the rows")
     if gate is not None:
         _rows(gate, "head_linear: gate")
-        if gate.dtype != x.dtype or gate.shape[0] != x.shape[0] or gate.shape[1] < H:
+        if gate.dtype != x.dtype or gate.shape[0] != x.shape[0] or gate.shape[1] < (H * n_out if gate_cols else H):
             raise KernelError("head_linear: the gate's rows do not fit the heads")
     call("mynah_head_linear_gated", ptr(x), ptr(W), ptr(out), code(x.dtype), x.shape[0], H, n_in, n_out,
          x.stride(0), head_in, in_off, out.stride(0), head_out, out_off, ptr(gate), gate.stride(0) if gate is not None else 0,
-         stream_ptr())
+         1 if gate_cols else 0, stream_ptr())
     return out
 
 
@@ -1037,15 +1069,19 @@ def moe_router_ffn(h: torch.Tensor, w_router: torch.Tensor, b_router: torch.Tens
 
 
 def rmsnorm_add(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, eps: float, extra: Optional[torch.Tensor] = None,
-                gain2: Optional[torch.Tensor] = None, eps2: float = 0.0) -> Optional[torch.Tensor]:
+                gain2: Optional[torch.Tensor] = None, eps2: float = 0.0, copy: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """x <- x (+ extra) + y / rms(y) * gain, all fp32 (csrc/norm_post.cu); with gain2 also returns the RMS norm of the
-    new x under gain2 and eps2 as fp32 rows."""
+    new x under gain2 and eps2 as fp32 rows. copy: bfloat16 rows that receive the new x, rounded."""
     _chk(x, "residual", torch.float32, 2)
     _chk(y, "sublayer output", torch.float32, 2)
     _chk(gain, "norm gain", dim=1)
     T, D = x.shape
     if y.shape != x.shape or gain.numel() != D or (extra is not None and (extra.shape != x.shape or extra.dtype != torch.float32)):
         raise KernelError("rmsnorm_add: shapes differ")
+    if copy is not None:
+        _chk(copy, "copy", torch.bfloat16, 2)
+        if copy.shape != x.shape:
+            raise KernelError("rmsnorm_add: the copy does not fit the rows")
     h = None
     if gain2 is not None:
         _chk(gain2, "second norm gain", dim=1)
@@ -1053,8 +1089,20 @@ def rmsnorm_add(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, eps: float
             raise KernelError("rmsnorm_add: the second gain does not fit the rows")
         h = torch.empty((T, D), dtype=torch.float32, device=x.device)
     call("mynah_rmsnorm_add", ptr(x), ptr(y), ptr(extra), ptr(gain), code(gain.dtype), float(eps), ptr(gain2),
-         code(gain2.dtype) if gain2 is not None else 0, float(eps2), ptr(h), T, D, stream_ptr())
+         code(gain2.dtype) if gain2 is not None else 0, float(eps2), ptr(h), ptr(copy), T, D, stream_ptr())
     return h
+
+
+def rms_rows(x: torch.Tensor, n: int, gain: torch.Tensor, eps: float) -> torch.Tensor:
+    """x[:, :n] / rms * gain as contiguous rows in x's type; x may be a column slice (csrc/norm_post.cu)."""
+    _rows(x, "rms_rows: input")
+    _chk(gain, "norm gain", dim=1)
+    if x.shape[1] < n or gain.numel() != n:
+        raise KernelError("rms_rows: the gain does not fit the rows")
+    out = torch.empty((x.shape[0], n), dtype=x.dtype, device=x.device)
+    call("mynah_rms_rows", ptr(x), code(x.dtype), max(x.stride(0), n), ptr(gain), code(gain.dtype), float(eps), ptr(out), n, x.shape[0], n,
+         stream_ptr())
+    return out
 
 
 def rms_pair_mean(a: torch.Tensor, b: torch.Tensor, ga: torch.Tensor, gb: torch.Tensor, eps: float,
@@ -1250,24 +1298,34 @@ def _out_rows(out: torch.Tensor, q: torch.Tensor, H: int, width: int) -> None:
         raise KernelError("attention output: the rows do not fit the heads")
 
 
+def _sink(sink: Optional[torch.Tensor], H: int):
+    if sink is not None:
+        _chk(sink, "sink", torch.float32, 1)
+        if sink.numel() != H:
+            raise KernelError(f"attention: {sink.numel()} sinks for {H} heads")
+    return ptr(sink)
+
+
 def attn_prefill_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int, k_cache, v_cache,
                         pages: PageTableView, window: int, scale: float, softcap: float, keep_first: int, vdiv: int,
-                        null_key: bool = False, out_scale: float = 1.0, vdo: Optional[int] = None) -> None:
+                        null_key: bool = False, out_scale: float = 1.0, vdo: Optional[int] = None,
+                        sink: Optional[torch.Tensor] = None) -> None:
     """The general prompt attention with capped scores, first tokens that the window keeps, `vdiv` key heads on one value
-    head, one more softmax term of score 0 without a value (null_key), a factor on the output, and output heads of `vdo`
-    columns (None: VD). `out` may be a column slice of wider rows."""
+    head, one more softmax term without a value, of score 0 (null_key) or of a score of its own for every query head (sink,
+    fp32 [H]; neither scaled nor capped), a factor on the output, and output heads of `vdo` columns (None: VD). `out` may be a column slice of wider rows."""
     _chk(q, "q", dim=2)
     _out_rows(out, q, H, VD if vdo is None else vdo)
     call("mynah_attn_prefill_generic_capped", ptr(q), ptr(out), code(q.dtype), q.shape[0], ctx.B, ctx.max_q_len, H, KV, HD, VD,
          q.shape[1], out.stride(0), ptr(k_cache), ptr(v_cache), ptr(ctx.cu_q), ptr(ctx.kv_len),
          ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages, window or 0, 0, float(scale), float(softcap or 0.0),
-         int(keep_first or 0), int(vdiv), 1 if null_key else 0, float(out_scale), int(vdo or 0), ptr(ctx.status), stream_ptr())
+         int(keep_first or 0), int(vdiv), 1 if null_key else 0, _sink(sink, H), float(out_scale), int(vdo or 0), ptr(ctx.status), stream_ptr())
 
 
 def attn_prefill_tcgen05_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, k_cache: torch.Tensor,
                                 v_cache: torch.Tensor, pages: PageTableView, window: int, scale: float, softcap: float,
                                 keep_first: int, vdiv: int, VD: Optional[int] = None, null_key: bool = False,
-                                out_scale: float = 1.0, vdo: Optional[int] = None) -> None:
+                                out_scale: float = 1.0, vdo: Optional[int] = None,
+                        sink: Optional[torch.Tensor] = None) -> None:
     """The tcgen05 prompt attention with capped scores, first tokens that the window keeps (the page lists must hold
     every page: a cache that gives pages back does not go with kept tokens) and `vdiv` key heads on one value head; value
     heads of VD columns (64 or 128; None: HD), a null key, an output factor and output heads of `vdo` columns (a multiple
@@ -1281,13 +1339,14 @@ def attn_prefill_tcgen05_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int,
     call("mynah_attn_prefill_tcgen05_capped", ptr(q), ptr(out), q.shape[0], ctx.B, ctx.max_q_len, H, KV, HD, q.stride(0),
          out.stride(0), ptr(k_cache), ptr(v_cache), ptr(ctx.cu_q), ptr(ctx.kv_len), ptr(pages.indptr), ptr(pages.ids),
          ptr(pages.base), pages.n_pages, window or 0, 0, float(scale), float(softcap or 0.0), int(keep_first or 0), int(vdiv),
-         int(VD or HD), 1 if null_key else 0, float(out_scale), int(vdo or VD or HD), ptr(ctx.status), stream_ptr())
+         int(VD or HD), 1 if null_key else 0, _sink(sink, H), float(out_scale), int(vdo or VD or HD), ptr(ctx.status), stream_ptr())
 
 
 def attn_decode_tc_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, k_cache: torch.Tensor,
                           v_cache: torch.Tensor, pages: PageTableView, window: int, scale: float, softcap: float,
                           keep_first: int, vdiv: int, scratch: torch.Tensor, VD: Optional[int] = None, null_key: bool = False,
-                          out_scale: float = 1.0, vdo: Optional[int] = None) -> None:
+                          out_scale: float = 1.0, vdo: Optional[int] = None,
+                        sink: Optional[torch.Tensor] = None) -> None:
     """The tensor-core decode attention with capped scores, first tokens that the window keeps (the page lists must hold
     every page) and `vdiv` key heads on one value head; the rest as in `attn_prefill_tcgen05_capped`."""
     VD = int(VD or HD)
@@ -1302,13 +1361,14 @@ def attn_decode_tc_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: i
     call("mynah_attn_decode_tc_capped", ptr(q), ptr(out), ctx.B, H, KV, HD, q.stride(0), out.stride(0),
          ptr(k_cache), ptr(v_cache), ptr(ctx.kv_len), ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages,
          window or 0, 0, float(scale), float(softcap or 0.0), int(keep_first or 0), int(vdiv), VD, 1 if null_key else 0,
-         float(out_scale), int(vdo or VD), ctx.decode_splits, ptr(scratch), None, ptr(ctx.status), stream_ptr())
+         _sink(sink, H), float(out_scale), int(vdo or VD), ctx.decode_splits, ptr(scratch), None, ptr(ctx.status), stream_ptr())
     lib.add_launches(1)        # pages and their merge
 
 
 def attn_decode_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int, HD: int, VD: int, k_cache, v_cache,
                        pages: PageTableView, window: int, scale: float, softcap: float, keep_first: int, vdiv: int,
-                       scratch: torch.Tensor, null_key: bool = False, out_scale: float = 1.0, vdo: Optional[int] = None) -> None:
+                       scratch: torch.Tensor, null_key: bool = False, out_scale: float = 1.0, vdo: Optional[int] = None,
+                        sink: Optional[torch.Tensor] = None) -> None:
     _chk(q, "q", dim=2)
     _out_rows(out, q, H, VD if vdo is None else vdo)
     _chk(scratch, "scratch", torch.float32)
@@ -1318,7 +1378,7 @@ def attn_decode_capped(q: torch.Tensor, out: torch.Tensor, ctx, H: int, KV: int,
     call("mynah_attn_decode_capped", ptr(q), ptr(out), code(q.dtype), ctx.B, H, KV, HD, VD, q.shape[1], out.stride(0),
          ptr(k_cache), ptr(v_cache), ptr(ctx.kv_len), ptr(pages.indptr), ptr(pages.ids), ptr(pages.base), pages.n_pages,
          window or 0, 0, float(scale), float(softcap or 0.0), int(keep_first or 0), int(vdiv), 1 if null_key else 0,
-         float(out_scale), int(vdo or 0), ctx.decode_splits, ptr(scratch), ptr(ctx.status), stream_ptr())
+         _sink(sink, H), float(out_scale), int(vdo or 0), ctx.decode_splits, ptr(scratch), ptr(ctx.status), stream_ptr())
     lib.add_launches(1)        # pages and their combination
 
 
@@ -1344,52 +1404,72 @@ def head_gate(x: torch.Tensor, gate: torch.Tensor, H: int, vd: int) -> torch.Ten
     return x
 
 
+def moe_runs_grouped(T: int, top: int, E: int, D: int, F: int, dtype: torch.dtype) -> bool:
+    """Whether a step of T tokens with `top` of E experts each runs its products as grouped tensor-core products."""
+    return int(lib.load().mynah_moe_grouped_rows(T, top, E, D, F, code(dtype))) > 0
+
+
 def moe_group_router_ffn(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], w_gu: torch.Tensor,
                          w_down: torch.Tensor, ctx, top: int, groups: int, keep: int, weight_scale: float,
                          limit: Optional[float], alpha: float, scores: str = "sigmoid", group_score: str = "top2",
-                         shared: Optional[torch.Tensor] = None) -> torch.Tensor:
+                         shared: Optional[torch.Tensor] = None, activation: str = "gated", weights_on: str = "output",
+                         shared_gate: bool = True, shared_expert: bool = False, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """Experts picked by sigmoid scores (fp32) with a correction for the choice, inside the `keep` best of `groups` groups of
     neighbouring experts; clamped-gate experts; weights score * weight_scale (csrc/moe.cu). w_router [E, D], correction
     [E] or None, w_gu [E, 2, F, D], w_down [E, D, F]; returns [T, D] in the rows' type. scores "softmax": over all
     experts; group_score "max": a group counts its largest. limit None: the experts' gate is silu(g) * u. shared: fp32
-    rows [T, D] of a shared expert, added times sigmoid of the product with one more row of w_router ([E + 1, D])."""
+    rows [T, D] of a shared expert, added times sigmoid of the product with one more row of w_router ([E + 1, D]), or as they
+    are (shared_gate False: w_router is [E, D]). activation "relu2": an expert is W_down relu(W_up h)^2, w_gu [E, F, D].
+    weights_on "input" (with relu2): a token's weight multiplies its expert's input instead of its output. shared_expert: the
+    last matrix of w_gu and w_down is a shared expert that every token passes with weight 1 (in place of `shared`). out_dtype
+    float32: the sum is not rounded to the rows' type."""
     _chk(h, "rows", dim=2)
     _chk(w_router, "router weights", h.dtype, 2)
     if correction is not None:
         _chk(correction, "router correction", dim=1)
     if scores not in ("sigmoid", "softmax") or group_score not in ("top2", "max"):
         raise KernelError("moe_group_router_ffn: unknown scores or group score")
-    _chk(w_gu, "gate/up weights", h.dtype, 4)
+    relu2 = activation == "relu2"
+    if activation not in ("gated", "relu2") or weights_on not in ("output", "input") or (weights_on == "input" and not relu2):
+        raise KernelError("moe_group_router_ffn: unknown activation, or weights on the input of gated experts")
+    _chk(w_gu, "up weights", h.dtype, 3 if relu2 else 4)
     _chk(w_down, "down weights", h.dtype, 3)
     T, D = h.shape
-    E, _, F, _ = w_gu.shape
-    rows = E + (1 if shared is not None else 0)
-    if (tuple(w_gu.shape) != (E, 2, F, D) or tuple(w_down.shape) != (E, D, F) or tuple(w_router.shape) != (rows, D)
+    n_mat, F = w_gu.shape[0], w_gu.shape[-2]
+    extra = 1 if shared_expert else 0
+    E = n_mat - extra
+    gated_rows = shared is not None and shared_gate
+    rows = E + (1 if gated_rows else 0)
+    if (tuple(w_gu.shape) != ((n_mat, F, D) if relu2 else (n_mat, 2, F, D)) or tuple(w_down.shape) != (n_mat, D, F)
+            or tuple(w_router.shape) != (rows, D) or (extra and (shared is not None or weights_on != "input"))
             or (correction is not None and correction.numel() != E) or not 1 <= top <= E):
         raise KernelError("moe_group_router_ffn: sizes do not fit")
     if shared is not None:
         _chk(shared, "shared expert's rows", torch.float32, 2)
         if shared.shape != h.shape:
             raise KernelError("moe_group_router_ffn: the shared expert's rows do not fit")
-    P_ = T * top
+    out_dtype = out_dtype or h.dtype
+    if out_dtype not in (h.dtype, torch.float32):
+        raise KernelError("moe_group_router_ffn: the result is in the rows' type or float32")
+    P_ = T * (top + extra)
     dev = h.device
-    grouped = int(lib.load().mynah_moe_grouped_rows(T, top, E, D, F, code(h.dtype)))
+    grouped = int(lib.load().mynah_moe_grouped_rows(T, top + extra, n_mat, D, F, code(h.dtype)))
     R = max(P_, grouped)
-    out = torch.empty((T, D), dtype=h.dtype, device=dev)
+    out = torch.empty((T, D), dtype=out_dtype, device=dev)
     y = torch.empty((R, F), dtype=h.dtype, device=dev)
     o = torch.empty((R, D), dtype=torch.float32, device=dev)
     a = torch.empty((R, D), dtype=h.dtype, device=dev) if grouped else None
-    ints = torch.empty((3 * P_ + 1 + 3 * int(lib.load().mynah_moe_max_tiles(T, top, E)) + R + R // 128 + 1,),
+    ints = torch.empty((3 * P_ + 1 + 3 * int(lib.load().mynah_moe_max_tiles(T, top + extra, n_mat)) + R + R // 128 + 1,),
                        dtype=torch.int32, device=dev)
     weights = torch.empty((P_ + T,), dtype=torch.float32, device=dev)         # the pairs' weights, then the shared expert's gates
     choice = ints[ints.numel() - P_:]
-    plain = limit is None
+    plain = limit is None or relu2
     call("mynah_moe_group_router_ffn", ptr(h), code(h.dtype), ptr(ctx.tok_seq), ptr(w_router), ptr(correction),
-         code(correction.dtype) if correction is not None else 0, ptr(w_gu), ptr(w_down), ptr(out), 0, ptr(y), ptr(o), ptr(ints),
+         code(correction.dtype) if correction is not None else 0, ptr(w_gu), ptr(w_down), ptr(out), 1 if out_dtype == torch.float32 else 0, ptr(y), ptr(o), ptr(ints),
          ptr(a), ptr(choice), ptr(weights), T, top, E, D, F, int(groups), int(keep), float(weight_scale),
          1 if scores == "softmax" else 0, 1 if group_score == "max" else 0, float("inf") if plain else float(limit),
-         1.0 if plain else float(alpha), 0.0 if plain else 1.0, ptr(shared), ptr(weights[P_:]) if shared is not None else None,
-         ptr(ctx.status), stream_ptr())
+         1.0 if plain else float(alpha), 0.0 if plain else 1.0, ptr(shared), ptr(weights[P_:]) if gated_rows else None,
+         2 if relu2 else 0, 1 if weights_on == "input" else 0, extra, ptr(ctx.status), stream_ptr())
     lib.add_launches(5 if grouped else 4)     # router, route, (gather,) two products, combine
     return out
 
@@ -1405,13 +1485,13 @@ def gated_memory(kind: str, p: torch.Tensor, at: dict, w2: Optional[torch.Tensor
                  q_scale: float, state: dict, out: torch.Tensor, ctx, H: int, dim: int, vd: int, eps: float, tau: float = 1.0,
                  cap: float = 1.0) -> torch.Tensor:
     """A recurrence with its output norm and gate (csrc/gated_memory.cu). kind "gla": decays per key channel from the narrow
-    row at["a"] (w2 [H * dim, rank], bias [H * dim], tau); "mlstm": input and forget gates at["i"], at["f"] (bias [2 H], cap). p:
-    the projection's rows; at: first columns of q, k, v, g and those. state: "S" [slots + 1, H, dim, vd], for "mlstm" also
+    row at["a"] (w2 [H * dim, rank], bias [H * dim], tau); "mlstm": input and forget gates at["i"], at["f"] (bias [2 H], cap);
+    "fixed": a decay a head (bias [2 H]: the decays, then their binary logarithms, finite). p: the projection's rows; at: first columns of q, k, v, g and those. state: "S" [slots + 1, H, dim, vd], for "mlstm" also
     "n" and "m", fp32. out: rows (a column slice is fine) whose first H * vd columns are written."""
     _rows(p, "gated_memory: projection")
     _rows(out, "gated_memory: output")
-    gla = kind == "gla"
-    if not gla and kind != "mlstm":
+    gla, fixed = kind == "gla", kind == "fixed"
+    if not gla and not fixed and kind != "mlstm":
         raise KernelError(f"gated_memory: unknown kind {kind!r}")
     S = state["S"]
     _chk(S, "memory state", torch.float32, 4)
@@ -1424,7 +1504,7 @@ def gated_memory(kind: str, p: torch.Tensor, at: dict, w2: Optional[torch.Tensor
         rank = w2.shape[1]
         if w2.shape[0] != H * dim or at["a"] + rank > p.shape[1]:
             raise KernelError("gated_memory: the decay's matrix does not fit the heads")
-    else:
+    elif not fixed:
         _chk(state["n"], "normaliser state", torch.float32, 3)
         _chk(state["m"], "stabiliser state", torch.float32, 2)
         if tuple(state["n"].shape[1:]) != (H, dim) or state["m"].shape[1] != H or max(at["i"], at["f"]) + H > p.shape[1]:
@@ -1434,11 +1514,12 @@ def gated_memory(kind: str, p: torch.Tensor, at: dict, w2: Optional[torch.Tensor
             or out.dtype != p.dtype or out.shape[0] != T or out.shape[1] < H * vd):
         raise KernelError("gated_memory: sizes do not fit")
     q_len = 1 if ctx.is_decode else int(ctx.max_q_len)
-    need = int(lib.load().mynah_gated_memory_scratch_floats(0 if gla else 1, code(p.dtype), T, ctx.B, H, dim, vd, rank, q_len))
+    number = {"gla": 0, "mlstm": 1, "fixed": 2}[kind]
+    need = int(lib.load().mynah_gated_memory_scratch_floats(number, code(p.dtype), T, ctx.B, H, dim, vd, rank, q_len))
     scratch = torch.empty((need,), dtype=torch.float32, device=p.device) if need else None
-    call("mynah_gated_memory", 0 if gla else 1, ptr(p), p.stride(0), at["q"], at["k"], at["v"], at["g"],
-         at["a"] if gla else at["i"], 0 if gla else at["f"], code(p.dtype), ptr(w2), rank, ptr(bias), ptr(w_norm), float(q_scale),
-         1.0 / float(tau), float(cap), float(eps), ptr(S), None if gla else ptr(state["n"]), None if gla else ptr(state["m"]),
+    call("mynah_gated_memory", number, ptr(p), p.stride(0), at["q"], at["k"], at["v"], at["g"],
+         0 if fixed else at["a"] if gla else at["i"], 0 if gla or fixed else at["f"], code(p.dtype), ptr(w2), rank, ptr(bias), ptr(w_norm), float(q_scale),
+         1.0 / float(tau), float(cap), float(eps), ptr(S), None if gla or fixed else ptr(state["n"]), None if gla or fixed else ptr(state["m"]),
          S.shape[0] - 1, ptr(out), out.stride(0), 0, ptr(ctx.cu_q), ptr(ctx.slots), ctx.B, T, H, dim, vd, q_len, ptr(scratch),
          stream_ptr())
     if need:

@@ -94,7 +94,7 @@ _SIGNATURES: dict[str, list] = {
                           c_int, c_int, c_int, c_int, c_int, c_int, c_int, P],
     "mynah_attn_prep": [P, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                         P, P, c_int, c_float, P, P, c_int, c_int, P, P, P, P, P, c_int,
-                        P, P, P, P, c_int, P, P],
+                        P, P, P, P, c_int, c_int, P, P],
     "mynah_attn_prefill_tcgen05_ex": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                       P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, P, P],
     "mynah_attn_decode_tc_ex": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P, P, P, P, P, c_int,
@@ -108,7 +108,9 @@ _SIGNATURES: dict[str, list] = {
     "mynah_delta_prep": [P, c_int, P, P, c_int, c_int, P, P, c_int, P, P, P, P, c_int, c_int, c_int, c_int, P, c_int, P],
     "mynah_delta_rule": [P, P, P, c_int, c_int, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, P],
     "mynah_gated_rmsnorm": [P, P, c_int, c_int, P, c_int, P, c_int, c_int, c_int, c_float, c_int, P],
-    "mynah_rmsnorm_add": [P, P, P, P, c_int, c_float, P, c_int, c_float, P, c_int, c_int, P],
+    "mynah_rmsnorm_add": [P, P, P, P, c_int, c_float, P, c_int, c_float, P, P, c_int, c_int, P],
+    "mynah_rms_rows": [P, c_int, c_int, P, c_int, c_float, P, c_int, c_int, c_int, P],
+    "mynah_embed_pairs": [P, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong, P, P],
     "mynah_rms_pair_mean": [P, P, P, P, c_int, c_float, c_float, P, c_int, c_int, P],
     "mynah_rglru_in": [P, c_int, c_int, c_int, c_int, P, P, c_int, P, P, c_int, c_int, P],
     "mynah_rglru_gates": [P, P, P, c_int, P, P, P, c_int, c_float, P, P, c_int, c_int, c_int, P],
@@ -125,19 +127,19 @@ _SIGNATURES: dict[str, list] = {
     "mynah_latent_prep": [P, c_int, c_int, P, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, c_int, c_int,
                           P, c_int, c_float, P, P, c_int, c_int, c_int, P, P, P, P, P, c_int, P, P, P],
     "mynah_head_linear": [P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P],
-    "mynah_head_linear_gated": [P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, c_int, P],
+    "mynah_head_linear_gated": [P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, c_int, c_int, P],
     "mynah_retention_prep": [P, c_int, c_int, c_int, c_int, P, P, c_int, c_int, c_int, P, P, c_int, c_int, c_int,
                              c_float, P, P, P, P],
     "mynah_retention_scan": [P, P, P, c_int, c_int, c_int, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P],
     "mynah_attn_prefill_tcgen05_capped": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_float, c_int,
+                                          P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, P, c_float, c_int,
                                           P, P],
     "mynah_attn_decode_tc_capped": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P, P, P, P, P, c_int,
-                                    c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_float, c_int, c_int, P, P, P, P],
+                                    c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, P, c_float, c_int, c_int, P, P, P, P],
     "mynah_attn_prefill_generic_capped": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_float, c_int, P, P],
+                                          P, P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, P, c_float, c_int, P, P],
     "mynah_attn_decode_capped": [P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                 P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_float, c_int,
+                                 P, P, P, P, P, P, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, P, c_float, c_int,
                                  c_int, P, P, P],
     "mynah_capped_attn_prep": [P, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                P, P, P, c_int, c_float, P, P, c_int, c_int, c_int, P, P, P, P, P, c_int, P, P, P, P, P],
@@ -145,7 +147,7 @@ _SIGNATURES: dict[str, list] = {
     "mynah_head_gate": [P, c_int, c_int, c_int, P, c_int, c_int, c_int, P],
     "mynah_residual_add_row": [P, P, c_longlong, c_int, P],
     "mynah_moe_group_router_ffn": [P, c_int, P, P, P, c_int, P, P, P, c_int, P, P, P, P, P, P, c_int, c_int, c_int, c_int,
-                                   c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_float, c_float, P, P, P, P],
+                                   c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_float, c_float, P, P, c_int, c_int, c_int, P, P],
     "mynah_softcap_f32": [P, c_longlong, c_float, P],
     "mynah_gated_memory": [c_int, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, c_int, P, P, c_float, c_float, c_float,
                            c_float, P, P, P, c_int, P, c_int, c_int, P, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P],

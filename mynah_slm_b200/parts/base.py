@@ -185,6 +185,14 @@ class FeedForward(Part):
 
 
 class Embedding(Part):
+    #: True for an embedding that also reads the step's context: forward(tokens, ctx)
+    needs_context = False
+
+    def state_request(self) -> Optional[StateRequest]:
+        """Per-sequence state of the embedding (the tokens before a step's first one, say), or None. With one,
+        forward is called as forward(tokens, ctx, state), state [max_seqs + 1, *shape] as in `CacheView.state`."""
+        return None
+
     def forward(self, tokens: torch.Tensor) -> torch.Tensor:
         """tokens: int32 [T] -> the first residual stream, fp32 [T, hidden]."""
         raise NotImplementedError
@@ -222,22 +230,27 @@ class Residual:
     delta that has not been added yet, with the constant it is multiplied by
     on its way in (1 unless a block scales its sublayers' outputs). A norm
     that follows an add takes both and does the add on its way (one pass over
-    the row instead of two)."""
+    the row instead of two). `rounded`, when a block has left it, is the stream
+    itself in the activation type (for a block that reads x as it is); every
+    change of the stream through this class drops it."""
 
     def __init__(self, x: torch.Tensor):
         self.x = x
         self.pending: Optional[torch.Tensor] = None
         self.pending_scale: float = 1.0
+        self.rounded: Optional[torch.Tensor] = None
 
     def add(self, delta: torch.Tensor, scale: float = 1.0) -> None:
         if self.pending is not None:
             self.flush()
+        self.rounded = None
         self.pending, self.pending_scale = delta, float(scale)
 
     def add_f32(self, delta: torch.Tensor) -> None:
         """Add fp32 rows now (after any pending delta): a sum that must not pass through the activation type."""
         from ..ops import kernels
         kernels.residual_add(self.flush(), delta, 1.0)
+        self.rounded = None
 
     def take_pending(self):
         """(delta, scale) of the add that is still to be done, which the caller now owes; (None, 1.0) if none."""

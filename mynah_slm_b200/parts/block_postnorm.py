@@ -54,18 +54,23 @@ class PostNormResidual(Block):
         return None
 
     def forward(self, stream: Residual, ctx, cache: CacheView) -> None:
-        x = stream.flush()
+        x, rounded = stream.flush(), stream.rounded
         if self.taps:
             state = cache.block_state["input_conv"] if self.taps > 1 else None
             h = kernels.causal_conv(x, self.conv_w, None, state, ctx, self.act_dtype, add_input=True)
         else:
-            h = x if self.act_dtype == torch.float32 else kernels.cast_rows(x, self.act_dtype)
+            h = x if self.act_dtype == torch.float32 else rounded if rounded is not None else kernels.cast_rows(x, self.act_dtype)
         y = self.mixer.forward(h, ctx, cache)
-        want_copy = self.ffn is not None and self.act_dtype != torch.float32
+        stream.rounded = None
+        # whoever reads x next wants it in the activation type: the feed-forward, or the next layer's mixer
+        reads_x = self.act_dtype != torch.float32 and not self.taps
+        want_copy = self.act_dtype != torch.float32 if self.ffn is not None else reads_x
         xc = self.norms["mixer"].add_normed(stream, y, copy=want_copy)
         if self.ffn is not None:
             y = self.ffn.forward(xc if xc is not None else stream.x, ctx)
-            self.norms["ffn"].add_normed(stream, y)
+            xc = self.norms["ffn"].add_normed(stream, y, copy=reads_x)
+        if reads_x:
+            stream.rounded = xc
 
 
 register_block("postnorm_residual", PostNormResidual)

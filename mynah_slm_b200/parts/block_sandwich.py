@@ -75,6 +75,7 @@ class SandwichResidual(Block):
 
     def forward(self, stream: Residual, ctx, cache: CacheView) -> None:
         x = stream.flush()
+        stream.rounded = None
         pre, post = self.norms["mixer"], self.norms["mixer_out"]
         h = kernels.rmsnorm(x, pre.gain, pre.eps, torch.float32)
         y = self.mixer.forward(self._input("mixer", h, ctx, cache), ctx, cache)

@@ -17,7 +17,7 @@ from typing import Mapping, Optional
 import torch
 
 from ..ops import kernels
-from .base import Embedding, Head, Part, TensorSpec, register_embedding, register_head
+from .base import Embedding, Head, Part, StateRequest, TensorSpec, register_embedding, register_head
 
 
 class TokenEmbedding(Embedding):
@@ -94,6 +94,38 @@ class TokenPositionEmbedding(Embedding):
 
 
 register_embedding("token_position_embedding", TokenPositionEmbedding)
+
+
+class TokenPairEmbedding(Embedding):
+    """x = E[token] + P[row]: a second table looked up by the token and the one before it, row = (token before * mul_prev
+    + token * mul_cur) mod buckets; a sequence's first token takes the table's last row (number `buckets`). Every
+    sequence's last token is kept as its state, so that a piece of a prompt or a decoded token finds the one before it.
+    Parameters: name, pair_name, vocab_size, dim, buckets, mul_prev, mul_cur."""
+    needs_context = True
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.name, self.pair_name = str(spec["name"]), str(spec["pair_name"])
+        self.V, self.D, self.buckets = int(spec["vocab_size"]), int(spec["dim"]), int(spec["buckets"])
+        # only the multipliers' remainders matter
+        self.mul_prev, self.mul_cur = int(spec["mul_prev"]) % self.buckets, int(spec["mul_cur"]) % self.buckets
+        self.table: Optional[torch.Tensor] = None
+        self.pairs: Optional[torch.Tensor] = None
+
+    def tensor_specs(self) -> list[TensorSpec]:
+        return [TensorSpec(self.name, (self.V, self.D)), TensorSpec(self.pair_name, (self.buckets + 1, self.D))]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], runtime) -> None:
+        self.table, self.pairs = tensors[self.name], tensors[self.pair_name]
+
+    def state_request(self):
+        return StateRequest((), torch.int32)
+
+    def forward(self, tokens: torch.Tensor, ctx, state: torch.Tensor) -> torch.Tensor:
+        return kernels.embed_pairs(self.table, self.pairs, state, ctx, self.mul_prev, self.mul_cur)
+
+
+register_embedding("token_pair_embedding", TokenPairEmbedding)
 
 
 class StreamVectors(Part):

@@ -4,7 +4,8 @@ x -> W_down . (silu(W_gate . x) * (W_up . x)), no bias (mynah-slm
 src/arch_qwen3.c:229-234, src/kernels.c:193-205). Parameters: hidden_size,
 intermediate_size, activation (only "silu" is built), and either prefix (the
 tensors are then <prefix>gate_proj.weight and so on) or the tensors' names gate,
-up and down. Gate and up are
+up and down; `output`: "act" (the default: rows in the run's activation type) or
+"fp32" (unrounded, for a norm that follows the sublayer). Gate and up are
 kept as one fused matrix [2 * intermediate, hidden], gate rows first, so a
 step is two products instead of three.
 """
@@ -33,6 +34,7 @@ class SwiGLUDense(FeedForward):
         act = spec.get("activation", "silu")
         if act != "silu":
             raise ConfigError(f"swiglu_dense: activation {act!r} is not supported (only 'silu')")
+        self.out_dtype = torch.float32 if str(spec.get("output", "act")) == "fp32" else None
         self.w_gate_up = self.w_down = None
 
     def tensor_specs(self) -> list[TensorSpec]:
@@ -48,7 +50,7 @@ class SwiGLUDense(FeedForward):
         return [self.w_gate_up, self.w_down]
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
-        return kernels.linear(kernels.linear_swiglu(h, self.w_gate_up), self.w_down)
+        return kernels.linear(kernels.linear_swiglu(h, self.w_gate_up), self.w_down, out_dtype=self.out_dtype)
 
 
 register_ffn("swiglu_dense", SwiGLUDense)

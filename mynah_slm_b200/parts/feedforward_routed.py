@@ -38,11 +38,15 @@ tensors are `<expert_prefix><e>.up` and `.down`.
 Variants, chosen by parameters: scores "softmax" (over all experts, instead of the sigmoid); group_score "max" (a group
 counts its largest choice score); correction None; limit None: the expert is W_down (silu(W_gate h) * (W_up h)). With
 `shared`, a feed-forward of that last form that every token passes (its intermediate size, and its tensors'
-`shared_prefix`), multiplied by sigmoid(w . h), one number a token (w: `shared_gate`), is added.
+`shared_prefix`), multiplied by sigmoid(w . h), one number a token (w: `shared_gate`; None: not multiplied), is added.
+activation "relu2": expert and shared expert are W_down relu(W_up h)^2 (`.up` and `.down`; no gate matrix). weights_on
+"input": a token's weight multiplies its expert's input instead of its output (one-matrix experts; the shared expert reads h as it
+is). Such a shared expert of the experts' own size runs as one more expert of small steps; else its two products are ordinary
+ones.
 
 Parameters: hidden_size, intermediate_size, experts, top, groups (1), keep (= groups), weight_scale (1), limit, alpha
-(1.702), scores ("sigmoid"), group_score ("top2"), router, correction (tensor names), expert_prefix, and optionally
-shared, shared_prefix, shared_gate.
+(1.702), scores ("sigmoid"), group_score ("top2"), activation ("gated"), weights_on ("output"), output ("act", or "fp32": the sum
+is not rounded), router, correction (tensor names), expert_prefix, and optionally shared, shared_prefix, shared_gate.
 """
 from __future__ import annotations
 
@@ -144,18 +148,27 @@ class GroupRouterExperts(FeedForward):
         self.groups = int(spec.get("groups", 1))
         self.keep = int(spec.get("keep", self.groups))
         self.weight_scale = float(spec.get("weight_scale", 1.0))
-        self.limit = None if spec["limit"] is None else float(spec["limit"])
+        self.limit = None if spec.get("limit") is None else float(spec["limit"])
         self.alpha = float(spec.get("alpha", 1.702))
         self.scores, self.group_score = str(spec.get("scores", "sigmoid")), str(spec.get("group_score", "top2"))
         self.router_name = str(spec["router"])
         self.correction_name = str(spec["correction"]) if spec.get("correction") is not None else None
         self.FS = int(spec.get("shared") or 0)
         self.shared_prefix = str(spec["shared_prefix"]) if self.FS else ""
-        self.shared_gate = str(spec["shared_gate"]) if self.FS else None
+        self.shared_gate = str(spec["shared_gate"]) if self.FS and spec.get("shared_gate") is not None else None
+        self.relu2 = str(spec.get("activation", "gated")) == "relu2"
+        self.weights_on = str(spec.get("weights_on", "output"))
+        self.out_dtype = torch.float32 if str(spec.get("output", "act")) == "fp32" else None
+        if spec.get("activation", "gated") not in ("gated", "relu2") or self.weights_on not in ("output", "input"):
+            raise ConfigError("group_router_experts: unknown activation or place of the weights")
+        if self.weights_on == "input" and not self.relu2:
+            raise ConfigError("group_router_experts: weights on the input go with experts of one matrix before the activation")
+        if self.relu2 and self.limit is not None:
+            raise ConfigError("group_router_experts: the squared relu has no limit")
         if self.scores not in ("sigmoid", "softmax") or self.group_score not in ("top2", "max"):
             raise ConfigError(f"group_router_experts: scores {self.scores!r} or group score {self.group_score!r} is not built in")
         self.prefix = str(spec["expert_prefix"])
-        if self.E > 1024:
+        if self.E + (1 if self.FS else 0) > 1024:
             raise ConfigError(f"group_router_experts: {self.E} experts exceed the 1024 that the routing kernel counts")
         if self.groups < 1 or self.E % self.groups or not 1 <= self.keep <= self.groups:
             raise ConfigError(f"group_router_experts: {self.E} experts do not form {self.groups} equal groups of which "
@@ -172,12 +185,18 @@ class GroupRouterExperts(FeedForward):
             specs.append(TensorSpec(self.correction_name, (self.E,), role="gain", init="normal", std=0.1))
         if self.FS:
             p = self.shared_prefix
-            specs += [TensorSpec(p + "gate", (self.FS, self.D)), TensorSpec(p + "up", (self.FS, self.D)),
-                      TensorSpec(p + "down", (self.D, self.FS)), TensorSpec(self.shared_gate, (1, self.D))]
+            specs += [TensorSpec(p + which, (self.FS, self.D)) for which in self._inner()]
+            specs.append(TensorSpec(p + "down", (self.D, self.FS)))
+            if self.shared_gate is not None:
+                specs.append(TensorSpec(self.shared_gate, (1, self.D)))
         for e in range(self.E):
-            specs += [TensorSpec(self._name(e, "gate"), (self.F, self.D)), TensorSpec(self._name(e, "up"), (self.F, self.D)),
-                      TensorSpec(self._name(e, "down"), (self.D, self.F))]
+            specs += [TensorSpec(self._name(e, which), (self.F, self.D)) for which in self._inner()]
+            specs.append(TensorSpec(self._name(e, "down"), (self.D, self.F)))
         return specs
+
+    def _inner(self) -> tuple[str, ...]:
+        """The matrices before the activation."""
+        return ("up",) if self.relu2 else ("gate", "up")
 
     def bind(self, tensors: Mapping[str, torch.Tensor], runtime) -> None:
         self.w_router = tensors[self.router_name].contiguous()
@@ -185,24 +204,38 @@ class GroupRouterExperts(FeedForward):
         self.w_shared = None
         if self.FS:
             p = self.shared_prefix
-            self.w_router = torch.cat([self.w_router, tensors[self.shared_gate]], dim=0).contiguous()
-            self.w_shared = torch.cat([tensors[p + "gate"], tensors[p + "up"]], dim=0).contiguous()
+            if self.shared_gate is not None:
+                self.w_router = torch.cat([self.w_router, tensors[self.shared_gate]], dim=0).contiguous()
+            self.w_shared = torch.cat([tensors[p + which] for which in self._inner()], dim=0).contiguous()
             self.w_shared_down = tensors[p + "down"]
-        self.w_gu = torch.stack([torch.stack([tensors[self._name(e, "gate")], tensors[self._name(e, "up")]])
-                                 for e in range(self.E)]).contiguous()
-        self.w_down = torch.stack([tensors[self._name(e, "down")] for e in range(self.E)]).contiguous()
+        names = [f"{self.prefix}{e}." for e in range(self.E)]
+        # a shared expert of the experts' own form and size, without a gate, lies behind them
+        self.shared_in_stack = bool(self.FS) and self.FS == self.F and self.weights_on == "input" and self.shared_gate is None
+        if self.shared_in_stack:
+            names.append(self.shared_prefix)
+        if self.relu2:
+            self.w_gu = torch.stack([tensors[n + "up"] for n in names]).contiguous()
+        else:
+            self.w_gu = torch.stack([torch.stack([tensors[n + "gate"], tensors[n + "up"]]) for n in names]).contiguous()
+        self.w_down = torch.stack([tensors[n + "down"] for n in names]).contiguous()
+        if self.shared_in_stack:                                 # one copy of it
+            self.w_shared, self.w_shared_down = self.w_gu[self.E], self.w_down[self.E]
 
     def streamed_tensors(self) -> list:
         # of the experts a step reads only those its tokens pick
         return [self.w_router] + ([self.w_shared, self.w_shared_down] if self.FS else [])
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
-        shared = None
-        if self.FS:
-            shared = kernels.linear(kernels.linear_swiglu(h, self.w_shared), self.w_shared_down, out_dtype=torch.float32)
-        return kernels.moe_group_router_ffn(h, self.w_router, self.correction, self.w_gu, self.w_down, ctx, self.top,
+        shared, w_gu, w_down = None, self.w_gu, self.w_down
+        in_stack = self.shared_in_stack and not kernels.moe_runs_grouped(h.shape[0], self.top + 1, self.E + 1, self.D, self.F, h.dtype)
+        if self.FS and not in_stack:
+            inner = kernels.linear_relu2 if self.relu2 else kernels.linear_swiglu
+            shared = kernels.linear(inner(h, self.w_shared), self.w_shared_down, out_dtype=torch.float32)
+            w_gu, w_down = w_gu[: self.E], w_down[: self.E]
+        return kernels.moe_group_router_ffn(h, self.w_router, self.correction, w_gu, w_down, ctx, self.top,
                                             self.groups, self.keep, self.weight_scale, self.limit, self.alpha, self.scores,
-                                            self.group_score, shared)
+                                            self.group_score, shared, "relu2" if self.relu2 else "gated", self.weights_on,
+                                            self.shared_gate is not None, in_stack, self.out_dtype)
 
 
 register_ffn("group_router_experts", GroupRouterExperts)

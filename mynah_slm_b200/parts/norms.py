@@ -6,7 +6,8 @@ src/kernels.c:118-128); the gain multiplies as it is, it is not 1 + w
 this one). That other function is here as a part of its own kind,
 `rmsnorm_offset`: out = x / sqrt(mean(x^2) + eps) * (1 + w); the sum 1 + w is
 formed once, in fp32, when the weights are bound. Parameters of both: eps,
-dim, and the gain's tensor name.
+dim, and the gain's tensor name. Either can stand behind a sublayer as well
+(`add_normed`).
 """
 from __future__ import annotations
 
@@ -39,6 +40,16 @@ class RMSNorm(Norm):
         if lazy and rows is None:
             return kernels.NormedInput(stream, delta, self.gain, self.eps, self.act_dtype, delta_scale=scale)
         return kernels.rmsnorm(stream.x, self.gain, self.eps, self.act_dtype, delta=delta, rows=rows, delta_scale=scale)
+
+    def add_normed(self, stream: Residual, y: torch.Tensor, copy: bool = False) -> Optional[torch.Tensor]:
+        """x <- x + norm(y) for fp32 rows y; with `copy` also returns the new x in the activation type."""
+        x = stream.flush()
+        if copy and self.act_dtype == torch.float32:
+            kernels.rmsnorm_add(x, y, self.gain, self.eps)
+            return x
+        c = torch.empty(x.shape, dtype=self.act_dtype, device=x.device) if copy else None
+        kernels.rmsnorm_add(x, y, self.gain, self.eps, copy=c)
+        return c
 
 
 class OffsetRMSNorm(RMSNorm):

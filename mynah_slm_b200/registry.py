@@ -94,6 +94,8 @@ def _register_builtin() -> None:
     register_architecture(gomuzen.ARCHITECTURE, gomuzen.GomuzenConfig.from_dict, replace=True)
     from .config import buludra
     register_architecture(buludra.ARCHITECTURE, buludra.BuludraConfig.from_dict, replace=True)
+    from .config import sagelorn
+    register_architecture(sagelorn.ARCHITECTURE, sagelorn.SagelornConfig.from_dict, replace=True)
 
 
 _register_builtin()
