@@ -10,6 +10,7 @@ and 64.
     python bench.py --design gupizen      (the Gupizen design beside Supisun, Nedupel and Qwen3 at equal size, likewise)
     python bench.py --design gomuzen      (the Gomuzen design beside Nedupel, Supisun and Qwen3 at equal size, likewise)
     python bench.py --design buludra      (the Buludra design beside Gupizen, Nedupel and Qwen3 at equal size, likewise)
+    python bench.py --design sagelorn     (the Sagelorn design beside Nedupel, Buludra and Qwen3 at equal size, likewise)
 
 One JSON line on stdout. A step is one decode step of the batch.
   value     decoded tokens per second, timed on the device with CUDA events
@@ -414,6 +415,32 @@ def buludra_config(shape: str, layers: int) -> dict:
             "logit_softcap": 15.0, "layers": [dict(pattern[i % 4], mlp=moe if i % 2 else dense) for i in range(layers)]}
 
 
+# The Sagelorn design at layer sizes that resemble a real model's, beside Nedupel (the closest existing design: retention,
+# latent attention, borrowed caches, experts), Buludra (experts beside a shared one) and Qwen3 at equal width, depth, heads
+# and vocabulary. Its layers repeat (attention, latent attention, attention that reads the keys of the one two layers
+# before, retention): the attentions keep the Qwen3 shape's heads with a window of 1,024 positions, a quarter of each head
+# rotated with scaled frequencies; the latent layers have a cache row of 96 + 32 values, queries through a latent of half
+# the width and the same window; retention has a state of head size x head size a head; feed-forwards alternate between
+# dense and 16 experts of half the dense width of which a token uses 2, beside a shared expert of the same size.
+def sagelorn_config(shape: str, layers: int) -> dict:
+    c = dict(QWEN3_0_6B)
+    c.update(SHAPES[shape])
+    D, H, G, HD, F = c["hidden_size"], c["num_attention_heads"], c["num_key_value_heads"], c["head_dim"], c["intermediate_size"]
+    dense = {"kind": "dense", "ff": F}
+    moe = {"kind": "moe", "expert": {"ff": F // 2}, "router": {"experts": 16, "top": 2}, "shared": {"ff": F // 2}}
+    att = {"heads": H, "kv_heads": G, "dim": HD, "vdim": HD, "scale": HD ** -0.5, "mask": {"size": 1024},
+           "rot": {"dims": HD // 4, "base": 1e6, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}}
+    lat = {"heads": H, "dim": HD - 32, "rot_dim": 32, "vdim": HD, "q_rank": D // 2, "kv_rank": 96, "scale": HD ** -0.5,
+           "rot": {"dims": 32, "base": 1e6}, "mask": {"size": 1024}}
+    ret = {"heads": H, "dim": HD, "vdim": HD, "decay": [1.0 - 2.0 ** (-5 - 3 * h / max(H - 1, 1)) for h in range(H)]}
+    out = []
+    for i in range(layers):
+        kind, m = [("attention", att), ("latent_attention", lat), ("attention", dict(att, kv_from=i - 2)), ("retention", ret)][i % 4]
+        out.append({"type": kind, "mixer": m, "mlp": moe if i % 2 else dense})
+    return {"architecture": "Sagelorn", "vocab": c["vocab_size"], "width": D, "max_positions": 8192, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}}, "logit_scale": 0.25, "layers": out}
+
+
 def run_design(args) -> int:
     """`--design NAME`: prefill of one 2,048-token prompt and decode steps at --batch behind 2,048-token prompts, for
     the design and for the existing models at equal size (`--model` runs one of them: for a launch list of that model alone)."""
@@ -445,6 +472,9 @@ def run_design(args) -> int:
         if args.design == "buludra":
             arms = [("buludra", buludra_config(shape, layers)), ("gupizen", gupizen_config(shape, layers)),
                     ("nedupel", nedupel_config(shape, layers)), ("qwen3", q)]
+        if args.design == "sagelorn":
+            arms = [("sagelorn", sagelorn_config(shape, layers)), ("nedupel", nedupel_config(shape, layers)),
+                    ("buludra", buludra_config(shape, layers)), ("qwen3", q)]
         for name, cfg in arms:
             if args.model and args.model != name:
                 continue
@@ -552,9 +582,9 @@ def main() -> int:
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="prompt length of the decode phases")
     ap.add_argument("--shape", default="0.6b", choices=sorted(SHAPES), help="layer sizes, for --only runs (the full line is always 0.6b)")
     ap.add_argument("--workload", default="", choices=["", "4b", "8b"], help="run one of the two larger workloads instead")
-    ap.add_argument("--design", default="", choices=["", "supisun", "nedupel", "gupizen", "gomuzen", "buludra"],
+    ap.add_argument("--design", default="", choices=["", "supisun", "nedupel", "gupizen", "gomuzen", "buludra", "sagelorn"],
                     help="measure this design beside Qwen3 at equal size instead (prefill and decode; a line of its own)")
-    ap.add_argument("--model", default="", choices=["", "supisun", "nedupel", "gupizen", "gomuzen", "buludra", "qwen3"], help="with --design: only this one of the models")
+    ap.add_argument("--model", default="", choices=["", "supisun", "nedupel", "gupizen", "gomuzen", "buludra", "sagelorn", "qwen3"], help="with --design: only this one of the models")
     args = ap.parse_args()
 
     if args.impl == "reference":
