@@ -344,6 +344,7 @@ moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecR
     const TA* x = h + (size_t)t * D;
     const int D8 = D % 8 == 0 ? D : 0;
     const int n_rows = shared_gate != nullptr ? E + 1 : E;           // the shared expert's gate is one more row
+    const bool by_logit = keep == groups || group_max;
     for (int e = warp; e < n_rows; e += (int)blockDim.x / 32) {
         const TA* wr = w + (size_t)e * D;
         float acc = 0.f;
@@ -365,7 +366,9 @@ moe_group_router_kernel(const TA* __restrict__ h, const TA* __restrict__ w, VecR
             } else {
                 const float s = 1.0f / (1.0f + expf(-acc));
                 sc[e] = s;
-                ch[e] = s + (correction.p != nullptr ? correction.at(e) : 0.f);
+                // without a correction (and without sums of scores) the choice goes by the logits: the same order, also where
+                // scores round to one
+                ch[e] = correction.p != nullptr ? s + correction.at(e) : (by_logit ? acc : s);
             }
         }
     }
