@@ -222,7 +222,7 @@ attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw
     float ss = 0.f;
 #pragma unroll
     for (int e = 0; e < 8; e++) ss = fmaf(x[e], x[e], ss);
-    const bool is_q = i < nq, is_k = !is_q && i < nq + nk, is_v = !is_q && !is_k && i < n_all;
+    const bool is_q = i < nq, is_k = !is_q && i < min(nq + nk, n_all), is_v = !is_q && !is_k && i < n_all;
     // q and k: two sums over the block, reduced together
     float sq = is_q ? ss : 0.f, sk = is_k ? ss : 0.f;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -329,7 +329,7 @@ MYNAH_API int mynah_attn_prep(const void* qkv, int dtype, int T, int ld, void* q
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     const VecRef qw{q_gain, gain_dtype}, kw{k_gain, gain_dtype};
     const int vd8 = vd / 8;
-    const bool v_lanes = !vnorm || ((vd8 & (vd8 - 1)) == 0 && vd8 <= 32 && ((H + G) * dim / 8) % vd8 == 0);
+    const bool v_lanes = !vnorm || (vd8 > 0 && (vd8 & (vd8 - 1)) == 0 && vd8 <= 32 && ((H + G) * dim / 8) % vd8 == 0);
     const bool one_phase = whole && vd % 8 == 0 && vdp % 8 == 0 && v_lanes && fits(v_cache) && fits(v_first) &&
                            H * dim + G * dim + G * vd <= 8 * 1024 &&
                            (dtype == MYNAH_F32 || dtype == MYNAH_BF16);
