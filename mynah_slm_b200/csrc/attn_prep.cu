@@ -20,6 +20,7 @@ struct PrepArgs {
     float eps;
     int vmix;        // 0: none, 1: write v_first, 2: mix with v_first
     int vnorm;       // 1: values are normed
+    int pairs_in_warp;   // 1: a head's pieces of eight lie inside one warp (see attn_prep_vec_kernel)
     int vec;         // 1: the q and k heads go eight elements a thread (see norm_rotate_heads8)
 };
 
@@ -180,121 +181,121 @@ attn_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw, Ve
     }
 }
 
-// The vector form of the whole kernel (taken when heads of q, k and v are whole 16-byte pieces, rot % 16 == 0 and a row has at
-// most 8 * 1024 elements; stored heads may be wider, the columns behind the head are zeros): a thread fetches its eight-element pieces of q, k and v at once, the three kinds of
-// sums of squares are formed together (q and k over the block, a value head that is normed over the lanes that hold it:
-// vd / 8, a power of two up to 32), and every piece is normed, rotated with its partner piece (fetched again from L1) and stored.
-template <typename T>
-__global__ void __launch_bounds__(1024)
+// The vector form of the whole kernel (taken when heads of q, k and v are whole 16-byte pieces, rot % 16 == 0 and q, and k and
+// v together, have at most 8 * 1024 elements; stored heads may be wider, the columns behind the head are zeros): one CTA takes the
+// queries of a row, another its keys and values, eight elements a thread; the sum of squares goes over the block (of a value head
+// that is normed over the lanes that hold it: vd / 8, a power of two up to 32), and every piece is normed, rotated with its
+// partner piece (another lane's, or fetched again from L1) and stored.
+template <typename T, int MAX_THREADS>
+__global__ void __launch_bounds__(MAX_THREADS)
 attn_prep_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, VecRef qw, VecRef kw,
                      const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                      const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, PageTable pt,
                      T* __restrict__ k_cache, T* __restrict__ v_cache, float* __restrict__ v_first,
                      const float* __restrict__ lambda_p, PrepArgs a, int* __restrict__ status) {
-    __shared__ float red[2][32];
-    griddep_launch_small();
-    griddep_wait();
+    __shared__ float red[32];
     const int row = blockIdx.x;
-    const int b = tok_seq[row];
     T* qo = q_out + (size_t)row * a.ldq;
     const int nq = a.H * a.dim, nk = a.G * a.dim, nv = a.G * a.vd;
-    const int i = threadIdx.x * 8;                 // this thread's piece of the row: q, then k, then v
-    const bool writes = k_cache != nullptr;
-    const int n_all = nq + (writes ? nk + nv : 0);
+    // this CTA's part of the row: q (blockIdx.y 0), or k and then v (1; not launched for a run that reads another run's cache)
+    const bool writes = blockIdx.y == 1;
+    const int i = (writes ? nq : 0) + threadIdx.x * 8;      // this thread's piece of the row
+    const int n_all = writes ? nq + nk + nv : nq;
+    const bool is_q = i < nq, is_k = writes && i < nq + nk, is_v = writes && !is_k && i < n_all;
+    // the gains of the piece, and everything else that needs no look-up, are on their way before the look-ups
+    const int local = is_q ? i : i - nq;           // index inside the projection (q and k)
+    const int h = local / a.dim, d = local - h * a.dim;
+    const VecRef gain{is_q ? qw.p : kw.p, qw.dtype};   // (one type for both)
+    float g[8] = {};
+    if (is_q || is_k) gain8(gain, local, g);
+    griddep_launch_small();
+    griddep_wait();
+    const T* src = qkv + (size_t)row * a.ld;
+    float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (i < n_all) load8(src + i, x);
+    const int b = tok_seq[row];
+    const int pos = tok_pos[row];
     if (b < 0) {
         float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        for (int j = i; j < a.H * a.dimp; j += blockDim.x * 8) store8(qo + j, zero);
+        if (!writes)
+            for (int j = i; j < a.H * a.dimp; j += blockDim.x * 8) store8(qo + j, zero);
         return;
     }
-    const int pos = tok_pos[row];
     if (a.rot > 0 && (pos < 0 || pos >= a.n_pos)) {
         if (threadIdx.x == 0) atomicOr(status, MYNAH_ST_POS_RANGE);
         return;
     }
+    // a rotated piece: its table entries, and where its partner piece lies
+    const int half = a.rot >> 1;
+    const bool turns = (is_q || is_k) && d < a.rot, low = d < half;
+    const int pd = low ? d + half : d - half;
+    float c[8], sn[8];
+    if (turns) {
+        load8(cos_t + (size_t)pos * half + (low ? d : pd), c);
+        load8(sin_t + (size_t)pos * half + (low ? d : pd), sn);
+    }
     const int page = writes ? page_of(pt, b, pos) : 0;
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; e++) ss = fmaf(x[e], x[e], ss);
+    const int lane = threadIdx.x & 31;
+    // a value head lies in vd / 8 consecutive threads of one warp (its start is a multiple of vd / 8 pieces)
+    float sv = ss;
+    if (a.vnorm) for (int o = (a.vd >> 3) >> 1; o > 0; o >>= 1) sv += __shfl_xor_sync(0xffffffffu, sv, o);
+    const float total = block_sum(is_q || is_k ? ss : 0.f, red);
     if (page < 0) {
         if (threadIdx.x == 0) atomicOr(status, MYNAH_ST_PAGE_RANGE);
         return;
     }
-    const T* src = qkv + (size_t)row * a.ld;
-    float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    if (i < n_all) load8(src + i, x);
-    float ss = 0.f;
-#pragma unroll
-    for (int e = 0; e < 8; e++) ss = fmaf(x[e], x[e], ss);
-    const bool is_q = i < nq, is_k = !is_q && i < min(nq + nk, n_all), is_v = !is_q && !is_k && i < n_all;
-    // q and k: two sums over the block, reduced together
-    float sq = is_q ? ss : 0.f, sk = is_k ? ss : 0.f;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    // a value head lies in vd / 8 consecutive threads of one warp (its start is a multiple of vd / 8 pieces)
-    float sv = ss;
-    if (a.vnorm) for (int o = (a.vd >> 3) >> 1; o > 0; o >>= 1) sv += __shfl_xor_sync(0xffffffffu, sv, o);
-    sq = warp_sum(sq);
-    sk = warp_sum(sk);
-    if (lane == 0) {
-        red[0][warp] = sq;
-        red[1][warp] = sk;
-    }
-    __syncthreads();
-    float tq = 0.f, tk = 0.f;
-    for (int w = 0; w < (int)(blockDim.x >> 5); w++) {
-        tq += red[0][w];
-        tk += red[1][w];
-    }
+    const float r = 1.0f / sqrtf(total / (float)(writes ? nk : nq) + a.eps);
     if (is_q || is_k) {
-        const float r = 1.0f / sqrtf((is_q ? tq / (float)nq : tk / (float)nk) + a.eps);
-        const int local = is_q ? i : i - nq;       // index inside the projection
-        const int h = local / a.dim, d = local % a.dim;
-        const VecRef& gain = is_q ? qw : kw;
-        float g[8], out[8];
-        gain8(gain, local, g);
 #pragma unroll
         for (int e = 0; e < 8; e++) x[e] = x[e] * r * g[e];
-        if (d < a.rot) {
-            const int half = a.rot >> 1;
-            const bool low = d < half;
-            const int pd = low ? d + half : d - half;          // the partner piece
-            float y[8], gy[8], c[8], sn[8];
-            load8(src + (is_q ? 0 : nq) + h * a.dim + pd, y);
-            gain8(gain, h * a.dim + pd, gy);
-            const float* cosr = cos_t + (size_t)pos * half + (low ? d : pd);
-            const float* sinr = sin_t + (size_t)pos * half + (low ? d : pd);
-            load8(cosr, c);
-            load8(sinr, sn);
+    }
+    float y[8];
+    if (a.pairs_in_warp) {                         // a head lies inside a warp: the partner is another lane's piece
+        const int from = turns ? (lane + (low ? half : -half) / 8) & 31 : lane;
 #pragma unroll
-            for (int e = 0; e < 8; e++) {
-                const float yy = y[e] * r * gy[e];
-                out[e] = low ? x[e] * c[e] - yy * sn[e] : x[e] * c[e] + yy * sn[e];
-            }
-        } else {
+        for (int e = 0; e < 8; e++) y[e] = __shfl_sync(0xffffffffu, x[e], from);
+    } else if (turns) {
+        float gy[8];
+        load8(src + (is_q ? 0 : nq) + h * a.dim + pd, y);
+        gain8(gain, h * a.dim + pd, gy);
 #pragma unroll
-            for (int e = 0; e < 8; e++) out[e] = x[e];
+        for (int e = 0; e < 8; e++) y[e] = y[e] * r * gy[e];
+    }
+    if (is_q || is_k) {
+        if (turns) {
+#pragma unroll
+            for (int e = 0; e < 8; e++) x[e] = low ? x[e] * c[e] - y[e] * sn[e] : x[e] * c[e] + y[e] * sn[e];
         }
-        if (is_q) store8(qo + h * a.dimp + d, out);
-        else store8(k_cache + (((size_t)page * a.G + h) * PAGE_TOKENS + pos % PAGE_TOKENS) * a.dimp + d, out);
+        if (is_q) store8(qo + h * a.dimp + d, x);
+        else store8(k_cache + (((size_t)page * a.G + h) * PAGE_TOKENS + pos % PAGE_TOKENS) * a.dimp + d, x);
     } else if (is_v) {
-        const int local = i - nq - nk;
-        const int g = local / a.vd, d = local % a.vd;
+        const int local_v = i - nq - nk;
+        const int gv = local_v / a.vd, dv = local_v % a.vd;
         const float rv = a.vnorm ? 1.0f / sqrtf(sv / (float)a.vd + a.eps) : 1.0f;
         float out[8];
 #pragma unroll
         for (int e = 0; e < 8; e++) out[e] = x[e] * rv;
         if (a.vmix == 1) {
-            store8(v_first + (size_t)row * nv + local, out);
+            store8(v_first + (size_t)row * nv + local_v, out);
         } else if (a.vmix == 2) {
             const float lam = *lambda_p;
             float f[8];
-            load8(v_first + (size_t)row * nv + local, f);
+            load8(v_first + (size_t)row * nv + local_v, f);
 #pragma unroll
             for (int e = 0; e < 8; e++) out[e] = (1.0f - lam) * out[e] + lam * f[e];
         }
-        store8(v_cache + (((size_t)page * a.G + g) * PAGE_TOKENS + pos % PAGE_TOKENS) * a.vdp + d, out);
+        store8(v_cache + (((size_t)page * a.G + gv) * PAGE_TOKENS + pos % PAGE_TOKENS) * a.vdp + dv, out);
     }
     // the columns behind the heads
     const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
     const int kp = (a.dimp - a.dim) >> 3, vp = (a.vdp - a.vd) >> 3;
-    for (int j = threadIdx.x; j < a.H * kp; j += blockDim.x) store8(qo + (j / kp) * a.dimp + a.dim + (j % kp) * 8, zero);
-    if (!writes) return;
+    if (!writes) {
+        for (int j = threadIdx.x; j < a.H * kp; j += blockDim.x) store8(qo + (j / kp) * a.dimp + a.dim + (j % kp) * 8, zero);
+        return;
+    }
     const size_t at = (size_t)page * a.G * PAGE_TOKENS + pos % PAGE_TOKENS;
     for (int j = threadIdx.x; j < a.G * kp; j += blockDim.x) store8(k_cache + (at + (size_t)(j / kp) * PAGE_TOKENS) * a.dimp + a.dim + (j % kp) * 8, zero);
     for (int j = threadIdx.x; j < a.G * vp; j += blockDim.x) store8(v_cache + (at + (size_t)(j / vp) * PAGE_TOKENS) * a.vdp + a.vd + (j % vp) * 8, zero);
@@ -325,23 +326,24 @@ MYNAH_API int mynah_attn_prep(const void* qkv, int dtype, int T, int ld, void* q
     const bool whole = dim % 8 == 0 && dimp % 8 == 0 && rot % 16 == 0 && ld % 8 == 0 && ldq % 8 == 0 && fits(qkv) && fits(q_out) &&
                        fits(q_gain) && fits(k_gain) && fits(cos_t) && fits(sin_t) && fits(k_cache);
     const int vec = whole && dimp == dim;
-    const PrepArgs a{H, G, dim, vd, dimp, vdp, ld, ldq, rot, n_pos, eps, vmix, vnorm, vec};
+    const PrepArgs a{H, G, dim, vd, dimp, vdp, ld, ldq, rot, n_pos, eps, vmix, vnorm, dim % 8 == 0 && 32 % (dim / 8) == 0, vec};
     const PageTable pt{page_indptr, page_ids, page_base, n_pages};
     const VecRef qw{q_gain, gain_dtype}, kw{k_gain, gain_dtype};
     const int vd8 = vd / 8;
-    const bool v_lanes = !vnorm || (vd8 > 0 && (vd8 & (vd8 - 1)) == 0 && vd8 <= 32 && ((H + G) * dim / 8) % vd8 == 0);
+    const bool v_lanes = !vnorm || (vd8 > 0 && (vd8 & (vd8 - 1)) == 0 && vd8 <= 32 && (G * dim / 8) % vd8 == 0);
     const bool one_phase = whole && vd % 8 == 0 && vdp % 8 == 0 && v_lanes && fits(v_cache) && fits(v_first) &&
-                           H * dim + G * dim + G * vd <= 8 * 1024 &&
+                           H * dim <= 8 * 1024 && G * (dim + vd) <= 8 * 1024 &&
                            (dtype == MYNAH_F32 || dtype == MYNAH_BF16);
     if (one_phase) {
-        const int n_all = H * dim + (k_cache ? G * (dim + vd) : 0);
-        const int threads = (n_all / 8 + 31) / 32 * 32;
-        if (dtype == MYNAH_F32)
-            mynah_launch(attn_prep_vec_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)qkv, (float*)q_out, qw, kw,
-                         cos_t, sin_t, tok_seq, tok_pos, pt, (float*)k_cache, (float*)v_cache, v_first, lambda_p, a, status);
-        else
-            mynah_launch(attn_prep_vec_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16*)qkv, (bf16*)q_out, qw, kw,
-                         cos_t, sin_t, tok_seq, tok_pos, pt, (bf16*)k_cache, (bf16*)v_cache, v_first, lambda_p, a, status);
+        const int n_kv = k_cache ? G * (dim + vd) : 0;
+        const int threads = ((H * dim > n_kv ? H * dim : n_kv) / 8 + 31) / 32 * 32;
+        auto go = [&](auto kern, auto zero) {
+            using T_ = decltype(zero);
+            mynah_launch(kern, dim3(T, k_cache ? 2 : 1), dim3(threads), 0, stream, (const T_*)qkv, (T_*)q_out, qw, kw, cos_t, sin_t, tok_seq, tok_pos, pt,
+                         (T_*)k_cache, (T_*)v_cache, v_first, lambda_p, a, status);
+        };
+        if (dtype == MYNAH_F32) threads <= 512 ? go(attn_prep_vec_kernel<float, 512>, float()) : go(attn_prep_vec_kernel<float, 1024>, float());
+        else threads <= 512 ? go(attn_prep_vec_kernel<bf16, 512>, bf16()) : go(attn_prep_vec_kernel<bf16, 1024>, bf16());
         return mynah_check_launch("attn_prep");
     }
     if (dtype == MYNAH_F32)

@@ -467,11 +467,18 @@ MYNAH_API int mynah_cast_f32(const float* in, void* out, int out_dtype, long lon
 
 // ----------------------------------------------------------------- scale
 // x[i] *= s in place (fp32): a head whose logits are multiplied by a constant.
+// four values a thread, in one 16-byte access where they are aligned
 __global__ void scale_f32_kernel(float* __restrict__ x, long long n, float s) {
     griddep_launch_small();
     griddep_wait();
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) x[i] *= s;
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (i + 3 < n && (reinterpret_cast<uintptr_t>(x) & 15) == 0) {
+        float4 v = *reinterpret_cast<const float4*>(x + i);
+        v.x *= s; v.y *= s; v.z *= s; v.w *= s;
+        *reinterpret_cast<float4*>(x + i) = v;
+        return;
+    }
+    for (long long j = i; j < n && j < i + 4; j++) x[j] *= s;
 }
 
 // x[i] = c tanh(x[i] / c) in place (fp32): a head whose logits are capped.
@@ -501,6 +508,6 @@ MYNAH_API int mynah_softcap_f32(float* x, long long n, float c, cudaStream_t str
 MYNAH_API int mynah_scale_f32(float* x, long long n, float s, cudaStream_t stream) {
     if (n == 0) return 0;
     MYNAH_REQUIRE(n > 0, "scale_f32: bad size %lld", n);
-    mynah_launch(scale_f32_kernel, dim3((unsigned)ceil_div_ll(n, 256)), dim3(256), 0, stream, x, n, s);
+    mynah_launch(scale_f32_kernel, dim3((unsigned)ceil_div_ll(n, 1024)), dim3(256), 0, stream, x, n, s);
     return mynah_check_launch("scale_f32");
 }

@@ -130,6 +130,7 @@ struct HeadLinearArgs {
     int ld_out, head_out, out_off;   // output likewise
     const void* gate;                // null, or rows in the activation type: head h's output is multiplied by
     int ld_gate;                     // sigmoid(gate[t * ld_gate + h]) on the accumulator, before it is rounded
+    int pairs;                       // 1: two neighbouring outputs (and their gates) lie in one aligned word
     int gate_cols;                   // 1: output column c of head h has a gate of its own, gate[t * ld_gate + h * n_out + c]
 };
 
@@ -197,6 +198,20 @@ head_linear_mma_kernel(const bf16* __restrict__ in, const bf16* __restrict__ W, 
     const bf16* wrow[1][NT];
 #pragma unroll
     for (int j = 0; j < NT; j++) wrow[0][j] = W + ((size_t)h * a.n_out + min(c0 + j * 8 + g, a.n_out - 1)) * a.n_in;
+    // a gate a value: the gates of this thread's outputs are on their way under the product
+    const bool early = a.gate_cols && a.pairs;
+    uint32_t gates[MT][2][NT];
+    if (early) {
+#pragma unroll
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+            for (int half = 0; half < 2; half++)
+#pragma unroll
+                for (int j = 0; j < NT; j++) {
+                    const int r = t0 + m * 16 + g + 8 * half, c = c0 + j * 8 + 2 * t;
+                    gates[m][half][j] = r < a.T && c < a.n_out ? *reinterpret_cast<const uint32_t*>(static_cast<const bf16*>(a.gate) + (size_t)r * a.ld_gate + (size_t)h * a.n_out + c) : 0u;
+                }
+    }
     float acc[1][MT][NT][4];
     tilemma::mma_tile<MT, NT, 1>(xs, row_s, in + (size_t)h * a.head_in + a.in_off, (size_t)a.ld_in, 1, wrow, a.n_in, acc);
 #pragma unroll
@@ -205,6 +220,20 @@ head_linear_mma_kernel(const bf16* __restrict__ in, const bf16* __restrict__ W, 
         for (int half = 0; half < 2; half++) {
             const int r = row_s[m * 16 + g + 8 * half];
             if (r < 0) continue;
+            if (a.pairs && (a.gate == nullptr || early)) {
+#pragma unroll
+                for (int j = 0; j < NT; j++) {
+                    const int c = c0 + j * 8 + 2 * t;
+                    if (c >= a.n_out) continue;
+                    float v0 = acc[0][m][j][2 * half], v1 = acc[0][m][j][2 * half + 1];
+                    if (early) {
+                        v0 *= 1.0f / (1.0f + expf(-__uint_as_float(gates[m][half][j] << 16)));
+                        v1 *= 1.0f / (1.0f + expf(-__uint_as_float(gates[m][half][j] & 0xffff0000u)));
+                    }
+                    *reinterpret_cast<__nv_bfloat162*>(out + (size_t)r * a.ld_out + (size_t)h * a.head_out + a.out_off + c) = __floats2bfloat162_rn(v0, v1);
+                }
+                continue;
+            }
             bf16* o = out + (size_t)r * a.ld_out + (size_t)h * a.head_out + a.out_off;
             const float gt = head_gate_of<bf16>(a, r, h);
 #pragma unroll
@@ -282,7 +311,9 @@ MYNAH_API int mynah_head_linear_gated(const void* in, const void* W, void* out, 
     if (T == 0) return 0;
     MYNAH_REQUIRE(T > 0 && H > 0 && n_in > 0 && n_out > 0, "head_linear: bad sizes");
     MYNAH_REQUIRE(H <= 65535 && ceil_div(n_out, 64) <= 65535, "head_linear: too many heads or outputs for one launch");
-    const HeadLinearArgs a{T, H, n_in, n_out, ld_in, head_in, in_off, ld_out, head_out, out_off, gate, ld_gate, gate_cols};
+    const HeadLinearArgs a{T, H, n_in, n_out, ld_in, head_in, in_off, ld_out, head_out, out_off, gate, ld_gate,
+                           (ld_out | head_out | out_off | n_out) % 2 == 0 && ((uintptr_t)out & 3) == 0 && (gate == nullptr || (ld_gate % 2 == 0 && ((uintptr_t)gate & 3) == 0)),
+                           gate_cols};
     const bool mma_ok = dtype == MYNAH_BF16 && !g_head_linear_plain && n_in % 8 == 0 && ld_in % 8 == 0 && head_in % 8 == 0 &&
                         in_off % 8 == 0 && (((uintptr_t)in | (uintptr_t)W) & 15) == 0 && ceil_div(n_out, 128) <= 65535;
     if (mma_ok) {

@@ -36,18 +36,10 @@ __device__ __forceinline__ void mma_tile(bf16 (*xs)[MMA_LDS], const int* row_s, 
 #pragma unroll
                 for (int e = 0; e < 4; e++) acc[s][m][j][e] = 0.f;
     for (int k0 = 0; k0 < K; k0 += MMA_KC) {
-        __syncthreads();
-        for (int idx = threadIdx.x; idx < 16 * MT * (MMA_KC / 8); idx += blockDim.x) {
-            const int r = idx / (MMA_KC / 8), kk = (idx % (MMA_KC / 8)) * 8;
-            const int p = row_s[r];
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (p >= 0 && k0 + kk < K) v = *reinterpret_cast<const uint4*>(src + (size_t)(p / src_div) * ld_src + k0 + kk);
-            *reinterpret_cast<uint4*>(&xs[r][kk]) = v;
-        }
-        __syncthreads();
         const int kend = min(MMA_KC, K - k0);
-        // the weights of the k-blocks after the ones being multiplied are already on their way: one block ahead under
-        // a tall tile (registers are the accumulators'), four under a 16-row tile (a decode step lives on loads in flight)
+        // the weights of the k-blocks after the ones being multiplied are already on their way (the first of them while the rows
+        // are staged): one block ahead under a tall tile (registers are the accumulators'), four under a 16-row tile (a decode
+        // step lives on loads in flight)
         constexpr int DEPTH = MT == 1 ? 4 : 1;
         auto fetch = [&](int kb, uint4 (&b)[DEPTH][NS][NT]) {
 #pragma unroll
@@ -63,6 +55,15 @@ __device__ __forceinline__ void mma_tile(bf16 (*xs)[MMA_LDS], const int* row_s, 
         };
         uint4 b[DEPTH][NS][NT], bn[DEPTH][NS][NT];
         fetch(0, b);
+        __syncthreads();
+        for (int idx = threadIdx.x; idx < 16 * MT * (MMA_KC / 8); idx += blockDim.x) {
+            const int r = idx / (MMA_KC / 8), kk = (idx % (MMA_KC / 8)) * 8;
+            const int p = row_s[r];
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (p >= 0 && k0 + kk < K) v = *reinterpret_cast<const uint4*>(src + (size_t)(p / src_div) * ld_src + k0 + kk);
+            *reinterpret_cast<uint4*>(&xs[r][kk]) = v;
+        }
+        __syncthreads();
         for (int kb = 0; kb < kend; kb += 32 * DEPTH) {
             fetch(kb + 32 * DEPTH, bn);                           // beyond the block: zeros, not used
 #pragma unroll
