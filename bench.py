@@ -438,7 +438,7 @@ def sagelorn_config(shape: str, layers: int) -> dict:
         kind, m = [("attention", att), ("latent_attention", lat), ("attention", dict(att, kv_from=i - 2)), ("retention", ret)][i % 4]
         out.append({"type": kind, "mixer": m, "mlp": moe if i % 2 else dense})
     return {"architecture": "Sagelorn", "vocab": c["vocab_size"], "width": D, "max_positions": 8192, "norm": {"eps": 1e-6},
-            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}}, "logit_scale": 0.25, "layers": out}
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 37, "mul_cur": 101}}, "logit_scale": 0.25, "layers": out}
 
 
 def run_design(args) -> int:

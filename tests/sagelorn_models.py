@@ -56,7 +56,7 @@ def bare(layer):
     return dict(layer, mlp=None)
 
 
-def config(width, vocab, layers, bigram=(97, 31, 17), eps=1e-5, logit_scale=0.7):
+def config(width, vocab, layers, bigram=(97, 29, 13), eps=1e-5, logit_scale=0.7):
     return {"architecture": "Sagelorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "logit_scale": logit_scale,
             "embedding": {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))}, "layers": layers}
 
@@ -99,9 +99,9 @@ SHARP = config(64, 150, [
 ], bigram=(1009, 37, 11))
 # widths that the tensor-core kernels take, as they are and padded to them; prompts longer than a tile
 WIDE = config(128, 257, [
-    moe(attention(4, 2, 64, 48, 0.15, rotation(16, 5000.0, (4.0, 1.0, 4.0, 200)), 100), 64, 8, 2, shared=64),
-    dense(latent(6, 32, 32, 32, 40, 64, 0.12, 3000.0, 70), 96),
-    moe(attention(4, 2, 64, 48, 0.13, rotation(16, 5000.0, (4.0, 1.0, 4.0, 200)), 250, kv_from=0), 72, 5, 1, shared=40),
+    moe(attention(6, 3, 64, 56, 0.15, rotation(32, 5000.0, (6.0, 1.0, 4.0, 200)), 100), 64, 8, 2, shared=64),
+    dense(latent(5, 40, 16, 32, 48, 72, 0.12, 3000.0, 70), 96),
+    moe(attention(6, 3, 64, 56, 0.13, rotation(32, 5000.0, (6.0, 1.0, 4.0, 200)), 250, kv_from=0), 72, 5, 1, shared=40),
     bare(retention(2, 64, 64, [0.98, 0.999])),
     dense(attention(3, 1, 128, 128, 0.1, rotation(128, 10000.0), 64), 64),
     bare(attention(2, 1, 100, 56, 0.1, rotation(32, 10000.0))),

@@ -99,7 +99,7 @@ def test_the_plain_implementation_notices_a_wrong_reading():
                         (("layers", 0, "mixer", "rot", "scaling", "factor"), 3.0), (("layers", 0, "mixer", "rot", "scaling", "high"), 6.0),
                         (("layers", 1, "mixer", "rot", "base"), 200.0), (("layers", 2, "mixer", "scale"), 0.42),
                         (("layers", 3, "mixer", "decay"), [0.9, 0.98, 0.995]), (("layers", 2, "mlp", "router", "top"), 2),
-                        (("logit_scale",), 0.71), (("embedding", "bigram", "mul_prev"), 30), (("embedding", "bigram", "buckets"), 96)):
+                        (("logit_scale",), 0.71), (("embedding", "bigram", "mul_prev"), 28), (("embedding", "bigram", "buckets"), 96)):
         assert rel_err(ref, _logits(_broken(path, value), W)) > 1e-3, path
     for name in ("l0.mix.sink", "l6.mix.sink", "l2.mix.q.norm", "l0.mix.k.norm", "l1.mix.dq.norm", "l1.mix.dkv.norm", "l1.mix.g",
                  "l3.norm1", "final.norm", "l1.mlp.router", "l1.mlp.shared.up", "l5.mlp.e1.down"):
@@ -137,11 +137,11 @@ def test_the_weight_stands_on_the_experts_input():
 
 def test_frequencies_against_the_rotation_part():
     from mynah_slm_b200.parts.position import rotary_frequencies
-    for dims, base, scaling in ((16, 500000.0, (4.0, 1.0, 4.0, 128)), (12, 500.0, (8.0, 0.5, 6.0, 60)), (8, 300.0, None)):
+    for dims, base, scaling in ((20, 400000.0, (3.0, 1.0, 4.0, 128)), (12, 500.0, (8.0, 0.5, 6.0, 60)), (8, 300.0, None)):
         rot = sm.rotation(dims, base, scaling)
         sc = {"kind": "wavelength", **rot["scaling"]} if scaling else None
         got, mult = rotary_frequencies(dims, base, sc)
         assert mult == 1.0 and np.allclose(got, plain.pair_frequencies(rot), rtol=1e-14)
-    f, f0 = plain.pair_frequencies(sm.rotation(16, 500000.0, (4.0, 1.0, 4.0, 128))), plain.pair_frequencies(sm.rotation(16, 500000.0))
-    kinds = {"kept": np.isclose(f, f0), "divided": np.isclose(f, f0 / 4.0)}
+    f, f0 = plain.pair_frequencies(sm.rotation(20, 400000.0, (3.0, 1.0, 4.0, 128))), plain.pair_frequencies(sm.rotation(20, 400000.0))
+    kinds = {"kept": np.isclose(f, f0), "divided": np.isclose(f, f0 / 3.0)}
     assert kinds["kept"].any() and kinds["divided"].any() and (~kinds["kept"] & ~kinds["divided"]).any()
